@@ -10,11 +10,27 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libbuddy_b200_kernels.so")
 
 F32, F16, BF16 = 0, 1, 2
-W_F32, W_I8, W_U4 = 0, 1, 2
+W_F32, W_I8, W_U4, W_BF16 = 0, 1, 2, 3
+MIX_LATENT = 0
+FF_NONE, FF_GATED, FF_EXPERTS = 0, 1, 2
 
 (T_EMBED, T_INV_FREQ, T_FINAL_NORM, T_LM_HEAD, T_IN_NORM, T_POST_NORM, T_Q_NORM,
  T_K_NORM, T_Q, T_K, T_V, T_O, T_GATE, T_UP, T_DOWN, T_Q_BIAS, T_K_BIAS,
  T_V_BIAS) = range(18)
+
+
+def build_if_missing():
+    """Compile the library in place when a checkout has none yet (one builder at a time)."""
+    import fcntl
+    import subprocess
+    if os.path.exists(LIB_PATH):
+        return
+    os.makedirs(os.path.join(_HERE, "csrc", "build"), exist_ok=True)
+    with open(os.path.join(_HERE, "csrc", "build", "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not os.path.exists(LIB_PATH):
+            subprocess.run(["make", "-C", os.path.join(_HERE, "csrc"), f"-j{os.cpu_count() or 4}"],
+                           check=True, stdout=subprocess.DEVNULL)
 
 
 class Weight(C.Structure):
@@ -38,6 +54,14 @@ class ModelConfigC(C.Structure):
                  "vocab", "max_len")] + \
                [("eps", C.c_float), ("rope_theta", C.c_float)] + \
                [(n, C.c_int32) for n in ("qkv_bias", "qk_norm", "tp_rank", "tp_size")]
+
+
+class LayerConfigC(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in
+                ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "kv_from")] + \
+               [("scale", C.c_float), ("rot_base", C.c_float)] + \
+               [(n, C.c_int32) for n in ("ff_kind", "ff", "experts", "top")] + \
+               [(n, C.c_float) for n in ("limit", "gate_slope", "up_offset")]
 
 
 class B200Error(RuntimeError):
@@ -92,6 +116,9 @@ def load():
         "b200_kv_overflow": (i32, [vp, i32, i32, i32, i32, i32, i32, f32,
                                    C.POINTER(C.c_int), vp]),
         "b200_model_create": (i32, [C.POINTER(ModelConfigC), C.POINTER(vp)]),
+        "b200_model_create_layered": (i32, [C.POINTER(ModelConfigC), C.POINTER(LayerConfigC), i32, C.POINTER(vp)]),
+        "b200_model_set_tensor": (i32, [vp, C.c_char_p, i32, vp, i64, i64]),
+        "b200_model_read_residual": (i32, [vp, vp, i32]),
         "b200_model_destroy": (None, [vp]),
         "b200_model_set_vector": (i32, [vp, i32, i32, vp, i64]),
         "b200_model_set_linear": (i32, [vp, i32, i32, i32, vp, vp, i32, i32, i64,
@@ -119,6 +146,7 @@ def load():
         "b200_batch_free_pages": (i32, [vp]),
         "b200_batch_prefill": (i32, [vp, i32, vp, i32, vp, C.POINTER(C.c_int)]),
         "b200_batch_decode": (i32, [vp, i32, vp, vp, vp, vp]),
+        "b200_batch_step": (i32, [vp, i32, vp, vp, vp, i32, vp, vp, vp]),
         "b200_batch_last_ms": (f32, [vp]),
         "b200_model_last_ms": (f32, [vp]),
         "b200_model_step_bytes": (i64, [vp, i32]),

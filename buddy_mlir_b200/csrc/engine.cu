@@ -10,8 +10,7 @@
 // parallel sharding follows examples/BuddyTensorParallel (column-parallel
 // q/k/v/gate/up, row-parallel o/down, sum after each, vocab-sharded lm_head;
 // buddy-deepseek-r1-distributed.cpp:521-617) with NCCL in place of MPI.
-#include "common.cuh"
-#include "mega.cuh"
+#include "engine.cuh"
 
 #include <dlfcn.h>
 
@@ -234,114 +233,11 @@ __global__ void advance_kernel(int32_t *token, int32_t *pos,
   }
 }
 
-struct DevLinear {
-  b200_weight w{};
-  void *w_buf = nullptr, *scale_buf = nullptr;
-  float *bias_buf = nullptr;
-  bool set = false;
-  int64_t bytes() const {
-    if (!set)
-      return 0;
-    int64_t b = packed_row_bytes(w.kind, w.K) * w.N;
-    if (w.scale) {
-      const int64_t ng =
-          (w.kind == B200_W_U4 && w.group > 0 && w.group < w.K) ? w.K / w.group : 1;
-      b += w.N * ng * (w.scale_dtype == B200_F32 ? 4 : 2);
-    }
-    if (w.bias)
-      b += w.N * 4;
-    return b;
-  }
-  void release() {
-    cudaFree(w_buf);
-    cudaFree(scale_buf);
-    cudaFree(bias_buf);
-    w_buf = scale_buf = nullptr;
-    bias_buf = nullptr;
-    set = false;
-  }
-};
-
-struct Layer {
-  float *in_norm = nullptr, *post_norm = nullptr, *q_norm = nullptr,
-        *k_norm = nullptr;
-  DevLinear q, k, v, o, gate, up, down;
-  DevLinear qkv, gateup;  // fused at finalize
-};
-
 } // namespace b200
 
 using namespace b200;
 
-struct b200_model {
-  b200_model_config cfg{};
-  int tp = 1, rank = 0;
-  int qh = 0, kvh = 0, ffn = 0, vocab = 0;  // local (sharded) sizes
-  float *embed = nullptr, *inv_freq = nullptr, *final_norm = nullptr;
-  std::vector<Layer> layers;
-  DevLinear lm_head;
-  std::vector<float *> kv;
-  float **kv_dev = nullptr;
-  float *x = nullptr, *qkv = nullptr, *attn = nullptr, *mid = nullptr,
-        *part = nullptr, *logits = nullptr, *logits_shard = nullptr;
-  float *attn_scratch = nullptr, *argmax_scratch = nullptr;
-  float *kv_stage = nullptr;  // [2*layers][kv_heads*D]: the rows written this step
-  int32_t *d_state = nullptr;  // token, pos, next, count, launches, -, error, -
-  int32_t *d_history = nullptr;
-  int history_cap = 0;
-  int splits = 1;
-  cudaStream_t stream = nullptr;
-  cudaGraph_t graph = nullptr;
-  cudaGraphExec_t exec = nullptr;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  float last_ms = 0.f;
-  int kernels_per_step = 0;
-  bool finalized = false;
-  float *h_logits_pinned = nullptr;
-  float *h_rows_pinned = nullptr;   // this step's K/V rows, fetched together with the logits
-  bool rows_fresh = false;
-  int32_t *h_state_pinned = nullptr;
-  // persistent decode-step kernel (batch 1, int8): see mega.cu
-  bool mega = false;
-  MegaParams mp{};
-  int mega_grid = 0;
-  size_t mega_smem = 0;
-  int64_t mega_stream_bytes = 0;
-  uint8_t *mega_stream = nullptr;
-  int64_t *mega_offsets = nullptr;   // [(4L+1)+1][grid]: per-phase and per-CTA stream offsets
-  const float **lvec_dev = nullptr;
-  uint2 *ll_buf = nullptr;           // tagged activation buffers
-  long long *d_trace = nullptr;
-  // prefill (many rows at once): activations of all rows, grown on demand
-  float *pf_x = nullptr, *pf_qkv = nullptr, *pf_att = nullptr, *pf_mid = nullptr, *pf_logits = nullptr;
-  float *pf_norm = nullptr;   // W8A8 only: the normalised rows of a projection
-  bool act_int8 = false;   // the w8a8 variant: int8 projections quantise their activations per call
-  uint32_t *q_row = nullptr;   // decode: the quantised activation row of the current projection
-  float *q_scale = nullptr;    //         and its scale
-  cudaGraph_t graph_q = nullptr;      // the decode step with int8 activations, captured on first use
-  cudaGraphExec_t exec_q = nullptr;
-  int kernels_per_step_q = 0;
-  void *pf_ws = nullptr;
-  int32_t *pf_tokens = nullptr;
-  int pf_rows = 0, pf_logit_rows = 0;
-  int64_t pf_ws_bytes = 0;
-  // tensor-parallel sums by peer stores (see TpPush): this rank's staging buffer and everybody's
-  uint2 *tp_ll = nullptr;
-  void *tp_opened[kTpMaxRanks] = {};
-  TpPush tp_push{};   // ranks == 0: the NCCL all-reduce is used instead
-  size_t tp_argmax_at = 0;   // pair offset of the (value, index) exchange slots inside the staging buffers
-};
-
 namespace {
-
-int dev_alloc(void **p, size_t bytes) {
-  cudaError_t e = cudaMalloc(p, bytes ? bytes : 16);
-  if (e != cudaSuccess) {
-    (void)cudaGetLastError();
-    return fail(B200_ENOMEM, "cudaMalloc(%zu): %s", bytes, cudaGetErrorString(e));
-  }
-  return B200_OK;
-}
 
 DevLinear *linear_slot(b200_model *m, int layer, int slot) {
   if (slot == B200_T_LM_HEAD)
@@ -490,8 +386,11 @@ int issue_step(b200_model *m, int *n_kernels) {
           *d_next = m->d_state + 2, *d_count = m->d_state + 3;
   cudaStream_t st = m->stream;
   const uint64_t before = b200_launch_count();
-  if (int rc = b200_embed(m->embed, d_token, m->x, H, st)) return rc;
-  for (int l = 0; l < c.n_layers; ++l) {
+  if (m->lay)
+    if (int rc = layered_issue_step(m, st)) return rc;
+  if (!m->lay)
+    if (int rc = b200_embed(m->embed, d_token, m->x, H, st)) return rc;
+  for (int l = 0; l < (int)m->layers.size(); ++l) {
     Layer &L = m->layers[l];
     float *q = m->qkv, *k = m->qkv + QD, *v = m->qkv + QD + KD;
     if (int rc = proj(m, L.qkv, m->x, m->qkv, nullptr, L.in_norm, false)) return rc;
@@ -517,7 +416,9 @@ int issue_step(b200_model *m, int *n_kernels) {
       if (int rc = gemv_tp_sum(m, L.down, m->mid, 2 * l + 1)) return rc;
     }
   }
-  if (m->tp == 1) {
+  if (m->lay) {
+    // its step ends with the logits
+  } else if (m->tp == 1) {
     if (int rc = proj(m, m->lm_head, m->x, m->logits, nullptr, m->final_norm, false))
       return rc;
   } else {
@@ -874,22 +775,32 @@ int b200_model_create(const b200_model_config *cfg, b200_model **out) {
                 "model_create: tp_size %d must divide kv_heads, q_heads, ffn and vocab", tp);
   if (tp > 1 && (!g_nccl.comm || g_nccl.size != tp || g_nccl.rank != c.tp_rank))
     return fail(B200_ESTATE, "model_create: call b200_tp_init(rank, size) first");
-  if (int rc = ensure_device()) return rc;
+  b200_model_config full = c;
+  full.tp_size = tp;
+  return model_allocate(full, out);
+}
 
+} // extern "C"
+
+// The handle of a session: streams, state words, per-step buffers and, for the uniform
+// attention layers (kv_heads > 0), their caches.
+int b200::model_allocate(const b200_model_config &c, b200_model **out) {
+  if (int rc = ensure_device()) return rc;
+  const int tp = c.tp_size;
   b200_model *m = new b200_model();
   m->cfg = c;
-  m->cfg.tp_size = tp;
   m->tp = tp;
   m->rank = c.tp_rank;
   m->qh = c.q_heads / tp;
   m->kvh = c.kv_heads / tp;
   m->ffn = c.ffn / tp;
   m->vocab = c.vocab / tp;
-  m->layers.resize(c.n_layers);
-  m->kv.assign(2 * c.n_layers, nullptr);
+  const bool uniform = c.kv_heads > 0;
+  m->layers.resize(uniform ? c.n_layers : 0);
+  m->kv.assign(uniform ? 2 * c.n_layers : 0, nullptr);
   const int D = c.head_dim;
   // attention splits: about four CTAs per SM over this rank's kv heads, at least 32 rows each
-  {
+  if (uniform) {
     const int local_kv = c.kv_heads / tp;
     m->splits = (4 * 148 + local_kv - 1) / local_kv;
     if (m->splits > c.max_len / 32) m->splits = c.max_len / 32;
@@ -921,7 +832,7 @@ int b200_model_create(const b200_model_config *cfg, b200_model **out) {
   A((void **)&m->kv_stage, (size_t)2 * c.n_layers * m->kvh * D * 4);
   A((void **)&m->d_state, 8 * sizeof(int32_t));
   A((void **)&m->d_history, m->history_cap * sizeof(int32_t));
-  if (rc == B200_OK &&
+  if (rc == B200_OK && uniform &&
       cudaMemcpy(m->kv_dev, m->kv.data(), m->kv.size() * sizeof(float *),
                  cudaMemcpyHostToDevice) != cudaSuccess)
     rc = fail(B200_ECUDA, "kv pointer table upload failed");
@@ -931,7 +842,7 @@ int b200_model_create(const b200_model_config *cfg, b200_model **out) {
     rc = fail(B200_ECUDA, "event create failed");
   if (rc == B200_OK && (cudaMallocHost((void **)&m->h_logits_pinned, (size_t)c.vocab * 4) != cudaSuccess ||
                         cudaMallocHost((void **)&m->h_rows_pinned,
-                                       (size_t)2 * c.n_layers * m->kvh * D * 4) != cudaSuccess ||
+                                       (size_t)2 * c.n_layers * m->kvh * D * 4 + 16) != cudaSuccess ||
                         cudaMallocHost((void **)&m->h_state_pinned, 32) != cudaSuccess))
     rc = fail(B200_ENOMEM, "pinned host allocation failed");
   if (rc != B200_OK) {
@@ -942,11 +853,14 @@ int b200_model_create(const b200_model_config *cfg, b200_model **out) {
   return B200_OK;
 }
 
+extern "C" {
+
 void b200_model_destroy(b200_model *m) {
   if (!m) return;
   if (m->stream) cudaStreamSynchronize(m->stream);
   if (m->exec) cudaGraphExecDestroy(m->exec);
   if (m->graph) cudaGraphDestroy(m->graph);
+  layered_destroy(m);
   for (auto &L : m->layers) {
     cudaFree(L.in_norm); cudaFree(L.post_norm); cudaFree(L.q_norm); cudaFree(L.k_norm);
     L.q.release(); L.k.release(); L.v.release(); L.o.release();
@@ -983,6 +897,8 @@ int b200_model_set_vector(b200_model *m, int layer, int slot, const float *host,
                           int64_t n) {
   if (!m || !host || n < 1)
     return fail(B200_EINVAL, "set_vector: bad argument");
+  if (m->lay)
+    return fail(B200_ESTATE, "set_vector: a model of described layers is loaded by b200_model_set_tensor");
   if (m->finalized)
     return fail(B200_ESTATE, "set_vector: model already finalised");
   const b200_model_config &c = m->cfg;
@@ -1035,6 +951,8 @@ int b200_model_set_linear(b200_model *m, int layer, int slot, int src_kind,
                           int quantize_to, int group) {
   if (!m || !host_w || K < 1 || N < 1)
     return fail(B200_EINVAL, "set_linear: bad argument");
+  if (m->lay)
+    return fail(B200_ESTATE, "set_linear: a model of described layers is loaded by b200_model_set_tensor");
   if (m->finalized)
     return fail(B200_ESTATE, "set_linear: model already finalised");
   DevLinear *L = linear_slot(m, layer, slot);
@@ -1200,6 +1118,8 @@ int b200_model_load_blobs(b200_model *m, const char *variant,
                           int all_linear_w8) {
   if (!m || !variant || !float_blob)
     return fail(B200_EINVAL, "load_blobs: null argument");
+  if (m->lay)
+    return fail(B200_ESTATE, "load_blobs: a model of described layers is loaded by b200_model_set_tensor");
   const b200_model_config &c = m->cfg;
   int64_t want_f = 0, want_i = 0;
   if (int rc = b200_blob_elements(&c, variant, &want_f, &want_i)) return rc;
@@ -1316,6 +1236,8 @@ int b200_model_load_blobs(b200_model *m, const char *variant,
 int b200_model_set_activation_int8(b200_model *m, int enabled) {
   if (!m)
     return fail(B200_EINVAL, "set_activation_int8: null model");
+  if (m->lay && enabled)
+    return fail(B200_ESTATE, "set_activation_int8: a model of described layers has no int8 projections");
   if (enabled && m->tp != 1)
     return fail(B200_ESTATE, "set_activation_int8: single-GPU sessions only");
   m->act_int8 = enabled != 0;
@@ -1473,6 +1395,8 @@ constexpr int kLinearSlots[] = {B200_T_Q, B200_T_K, B200_T_V, B200_T_O, B200_T_G
 int b200_model_save_packed(b200_model *m, const char *path) {
   if (!m || !path)
     return fail(B200_EINVAL, "save_packed: null argument");
+  if (m->lay)
+    return fail(B200_ESTATE, "save_packed: a model of described layers is loaded from its own tensors");
   if (m->finalized)
     return fail(B200_ESTATE, "save_packed: call it before finalize (finalize frees the per-projection buffers)");
   FILE *f = fopen(path, "wb");
@@ -1531,6 +1455,8 @@ int b200_model_save_packed(b200_model *m, const char *path) {
 int b200_model_load_packed(b200_model *m, const char *path) {
   if (!m || !path)
     return fail(B200_EINVAL, "load_packed: null argument");
+  if (m->lay)
+    return fail(B200_ESTATE, "load_packed: a model of described layers is loaded from its own tensors");
   if (m->finalized)
     return fail(B200_ESTATE, "load_packed: model already finalised");
   FILE *f = fopen(path, "rb");
@@ -1588,16 +1514,18 @@ int b200_model_finalize(b200_model *m) {
   if (m->finalized)
     return B200_OK;
   const b200_model_config &c = m->cfg;
-  if (!m->embed || !m->final_norm || !m->lm_head.set)
+  if (m->lay) {
+    if (int rc = layered_ready(m)) return rc;
+  } else if (!m->embed || !m->final_norm || !m->lm_head.set)
     return fail(B200_ESTATE, "finalize: embedding, final norm or lm_head missing");
-  if (!m->inv_freq) {
+  if (!m->inv_freq && !m->lay) {
     std::vector<float> f(c.head_dim / 2);
     for (int j = 0; j < c.head_dim / 2; ++j)
       f[j] = (float)(1.0 / std::pow((double)c.rope_theta, (2.0 * j) / c.head_dim));
     if (int rc = b200_model_set_vector(m, -1, B200_T_INV_FREQ, f.data(), f.size()))
       return rc;
   }
-  for (int l = 0; l < c.n_layers; ++l) {
+  for (int l = 0; l < (int)m->layers.size(); ++l) {
     Layer &L = m->layers[l];
     if (!L.in_norm || !L.post_norm || !L.q.set || !L.k.set || !L.v.set ||
         !L.o.set || !L.gate.set || !L.up.set || !L.down.set)
@@ -1608,7 +1536,7 @@ int b200_model_finalize(b200_model *m) {
     if (int rc = fuse_linears({&L.gate, &L.up}, true, &L.gateup, m->stream)) return rc;
     L.q.release(); L.k.release(); L.v.release();
   }
-  if (mega_eligible(m, m->layers[0]))
+  if (!m->lay && mega_eligible(m, m->layers[0]))
     if (int rc = build_mega(m)) return rc;
   for (auto &L : m->layers) { L.gate.release(); L.up.release(); }
   if (m->mega) {
@@ -1641,6 +1569,8 @@ int b200_model_finalize(b200_model *m) {
   B200_CUDA(cudaStreamSynchronize(m->stream));
   for (auto p : m->kv)  // the warm-up wrote row 0
     B200_CUDA(cudaMemsetAsync(p, 0, (size_t)m->kvh * c.max_len * c.head_dim * 4, m->stream));
+  if (m->lay)
+    if (int rc = layered_clear_cache(m)) return rc;
   B200_CUDA(cudaStreamBeginCapture(m->stream, cudaStreamCaptureModeThreadLocal));
   int rc = issue_step(m, nullptr);
   cudaGraph_t g = nullptr;
@@ -1851,6 +1781,29 @@ int b200_model_prefill(b200_model *m, const int32_t *tokens, int n_tokens, int p
     if (tokens[i] < 0 || tokens[i] >= c.vocab)
       return fail(B200_EINVAL, "prefill: token %d at row %d out of range", tokens[i], i);
   const int M = n_tokens, D = c.head_dim, H = c.hidden;
+  if (m->lay) {
+    // the session's cache is one page of max_len positions of one sequence
+    std::vector<int32_t> rs((size_t)M, 0), rp((size_t)M), want;
+    std::vector<void *> pools;
+    for (auto &L : m->lay->layers)
+      pools.push_back(L.cache);
+    for (int i = 0; i < M; ++i)
+      rp[(size_t)i] = pos0 + i;
+    for (int i = all_rows && logits_host ? 0 : M - 1; i < M; ++i)
+      want.push_back(i);
+    std::vector<int32_t> nxt(want.size());
+    B200_CUDA(cudaEventRecord(m->ev0, m->stream));
+    if (int rc = layered_rows(m, M, tokens, rs.data(), rp.data(), m->lay->zero, 1, c.max_len, pools.data(), c.max_len,
+                              (int)want.size(), want.data(), logits_host, nxt.data()))
+      return rc;
+    B200_CUDA(cudaEventRecord(m->ev1, m->stream));
+    B200_CUDA(cudaStreamSynchronize(m->stream));
+    B200_CUDA(cudaEventElapsedTime(&m->last_ms, m->ev0, m->ev1));
+    m->rows_fresh = false;
+    if (next_token)
+      *next_token = nxt.back();
+    return B200_OK;
+  }
   const int64_t QD = (int64_t)m->qh * D, KD = (int64_t)m->kvh * D, QKV = QD + 2 * KD;
   // w8a8: the activation scale of the last projection belongs to all rows, so all of them are computed
   const int logit_rows = ((all_rows && logits_host) || m->act_int8) ? M : 1;
@@ -1901,23 +1854,21 @@ int b200_model_prefill(b200_model *m, const int32_t *tokens, int n_tokens, int p
 }
 
 // ---- batched decode over a paged KV cache ------------------------------------------------
-struct b200_batch {
-  b200_model *m = nullptr;
-  int max_seqs = 0, page = 0, n_pages = 0, table_stride = 0;
-  std::vector<float *> pool;            // [2 * layers] page pools [n_pages][kv_heads][page][D]
-  std::vector<int> free_pages;
-  std::vector<int> len;                 // per sequence: -1 = unused slot
-  std::vector<int32_t> table;           // [max_seqs][table_stride] host mirror
-  int32_t *d_table = nullptr, *d_seq = nullptr, *d_pos = nullptr, *d_next = nullptr;
-  float *d_part = nullptr;              // attention partials of the key-split scan, for up to part_rows rows
-  int part_rows = 0, max_context = 0;
-  int rows_cap = 0;
-  float last_ms = 0.f;
-};
-
 static int batch_rows(b200_batch *b, int M, const int32_t *tokens, const int32_t *row_seq, const int32_t *row_pos,
-                      bool all_logits, float *logits_host, int32_t *next_host) {
+                      int n_want, const int32_t *want, float *logits_host, int32_t *next_host) {
   b200_model *m = b->m;
+  if (m->lay) {
+    cudaStream_t st = m->stream;
+    B200_CUDA(cudaMemcpyAsync(b->d_table, b->table.data(), b->table.size() * 4, cudaMemcpyHostToDevice, st));
+    B200_CUDA(cudaEventRecord(m->ev0, st));
+    if (int rc = layered_rows(m, M, tokens, row_seq, row_pos, b->d_table, b->table_stride, b->page, b->rows_pool.data(),
+                              b->max_context, n_want, want, logits_host, next_host))
+      return rc;
+    B200_CUDA(cudaEventRecord(m->ev1, st));
+    B200_CUDA(cudaStreamSynchronize(st));
+    B200_CUDA(cudaEventElapsedTime(&b->last_ms, m->ev0, m->ev1));
+    return B200_OK;
+  }
   // A w8a8 projection scales its whole activation tensor: rows of unrelated sequences in one
   // batch would share that scale, and each sequence's result would depend on its neighbours.
   if (m->act_int8)
@@ -1925,8 +1876,8 @@ static int batch_rows(b200_batch *b, int M, const int32_t *tokens, const int32_t
   const b200_model_config &c = m->cfg;
   const int D = c.head_dim, H = c.hidden;
   const int64_t QD = (int64_t)m->qh * D, KD = (int64_t)m->kvh * D, QKV = QD + 2 * KD;
-  const int logit_rows = all_logits ? M : 1;
-  if (int rc = prefill_reserve(m, M, logit_rows)) return rc;
+  const int logit_rows = n_want;
+  if (int rc = prefill_reserve(m, M, logit_rows > 0 ? logit_rows : 1)) return rc;
   cudaStream_t st = m->stream;
   if (M > b->rows_cap) {
     cudaFree(b->d_seq); cudaFree(b->d_pos); cudaFree(b->d_next);
@@ -1968,15 +1919,28 @@ static int batch_rows(b200_batch *b, int M, const int32_t *tokens, const int32_t
     if (int rc = linear_rows(m, L.gateup, m->pf_x, H, M, m->pf_mid, m->ffn, nullptr, L.post_norm, true)) return rc;
     if (int rc = linear_rows(m, L.down, m->pf_mid, m->ffn, M, m->pf_x, H, m->pf_x, nullptr, false)) return rc;
   }
-  const int first = all_logits ? 0 : M - 1;
-  if (int rc = linear_rows(m, m->lm_head, m->pf_x + (int64_t)first * H, H, logit_rows, m->pf_logits, c.vocab, nullptr,
-                           m->final_norm, false))
-    return rc;
-  if (int rc = argmax_rows_launch(m->pf_logits, c.vocab, logit_rows, b->d_next, st)) return rc;
+  if (n_want > 0) {
+    // the wanted rows move up (their order is ascending, so a row is read before it is overwritten)
+    int first = want[0];
+    bool run = true;
+    for (int i = 1; i < n_want; ++i)
+      run = run && want[i] == first + i;
+    if (!run) {
+      for (int i = 0; i < n_want; ++i)
+        if (want[i] != i)
+          B200_CUDA(cudaMemcpyAsync(m->pf_x + (int64_t)i * H, m->pf_x + (int64_t)want[i] * H, (size_t)H * 4,
+                                    cudaMemcpyDeviceToDevice, st));
+      first = 0;
+    }
+    if (int rc = linear_rows(m, m->lm_head, m->pf_x + (int64_t)first * H, H, logit_rows, m->pf_logits, c.vocab, nullptr,
+                             m->final_norm, false))
+      return rc;
+    if (int rc = argmax_rows_launch(m->pf_logits, c.vocab, logit_rows, b->d_next, st)) return rc;
+  }
   B200_CUDA(cudaEventRecord(m->ev1, st));
-  if (logits_host)
+  if (logits_host && n_want > 0)
     B200_CUDA(cudaMemcpyAsync(logits_host, m->pf_logits, (size_t)logit_rows * c.vocab * 4, cudaMemcpyDeviceToHost, st));
-  if (next_host)
+  if (next_host && n_want > 0)
     B200_CUDA(cudaMemcpyAsync(next_host, b->d_next, (size_t)logit_rows * 4, cudaMemcpyDeviceToHost, st));
   B200_CUDA(cudaStreamSynchronize(st));
   B200_CUDA(cudaEventElapsedTime(&b->last_ms, m->ev0, m->ev1));
@@ -1998,6 +1962,25 @@ static int batch_grow(b200_batch *b, int seq, int n) {
   return B200_OK;
 }
 
+// The reverse of batch_grow for a step that did not run.
+static void batch_ungrow(b200_batch *b, int seq, int n) {
+  const int have = (b->len[seq] + b->page - 1) / b->page, want = (b->len[seq] + n + b->page - 1) / b->page;
+  for (int i = want - 1; i >= have; --i)
+    b->free_pages.push_back(b->table[(size_t)seq * b->table_stride + i]);
+}
+
+// A sequence has grown to len positions: pages that no layer's window reaches any more go back to
+// the free list (only where every layer has a window; the next position sees window - 1 before it).
+static void batch_release_passed(b200_batch *b, int seq) {
+  const int window = b->m->lay ? b->m->lay->window : 0;
+  if (window <= 0)
+    return;
+  while ((b->first[seq] + 1) * b->page <= b->len[seq] - window + 1) {
+    b->free_pages.push_back(b->table[(size_t)seq * b->table_stride + b->first[seq]]);
+    b->first[seq] += 1;
+  }
+}
+
 int b200_batch_create(b200_model *m, int max_seqs, int page_size, int n_pages, int max_context, b200_batch **out) {
   if (!m || !out || max_seqs < 1 || page_size < 1 || n_pages < 1 || max_context < 1)
     return fail(B200_EINVAL, "batch_create: bad argument");
@@ -2013,18 +1996,33 @@ int b200_batch_create(b200_model *m, int max_seqs, int page_size, int n_pages, i
   b->table.assign((size_t)max_seqs * b->table_stride, 0);
   for (int i = n_pages - 1; i >= 0; --i)
     b->free_pages.push_back(i);
+  b->first.assign(max_seqs, 0);
   const size_t pool_bytes = (size_t)n_pages * m->kvh * page_size * m->cfg.head_dim * 4;
-  b->pool.assign(2 * m->cfg.n_layers, nullptr);
+  b->pool.assign(m->kv.size(), nullptr);
   int rc = B200_OK;
   for (auto &p : b->pool)
     if (rc == B200_OK) rc = dev_alloc((void **)&p, pool_bytes);
+  if (m->lay) {
+    const size_t e = m->lay->dtype == B200_F32 ? 4 : 2;
+    for (auto &L : m->lay->layers) {
+      void *p = nullptr;
+      const size_t bytes = (size_t)n_pages * page_size * L.d.row * e;
+      if (rc == B200_OK && L.own()) {
+        rc = dev_alloc(&p, bytes);
+        // padding elements of a row are read and never written
+        if (rc == B200_OK && cudaMemset(p, 0, bytes) != cudaSuccess)
+          rc = fail(B200_ECUDA, "batch_create: cudaMemset failed");
+      }
+      b->rows_pool.push_back(L.own() ? p : b->rows_pool[(size_t)L.source]);
+    }
+  }
   if (rc == B200_OK) rc = dev_alloc((void **)&b->d_table, b->table.size() * 4);
   b->max_context = b->table_stride * page_size;
   b->part_rows = max_seqs;
-  if (rc == B200_OK)
+  if (rc == B200_OK && !m->lay)
     rc = dev_alloc((void **)&b->d_part,
                    (size_t)gqa_paged_scratch_floats(b->part_rows, m->qh, m->cfg.head_dim, b->max_context) * 4);
-  if (rc == B200_OK && cudaMemset(b->d_part, 0, (size_t)b->part_rows * m->qh * 4) != cudaSuccess)   // the counters
+  if (rc == B200_OK && !m->lay && cudaMemset(b->d_part, 0, (size_t)b->part_rows * m->qh * 4) != cudaSuccess)   // the counters
     rc = fail(B200_ECUDA, "batch_create: cudaMemset failed");
   if (rc != B200_OK) {
     b200_batch_destroy(b);
@@ -2037,6 +2035,8 @@ int b200_batch_create(b200_model *m, int max_seqs, int page_size, int n_pages, i
 void b200_batch_destroy(b200_batch *b) {
   if (!b) return;
   for (auto p : b->pool) cudaFree(p);
+  for (size_t i = 0; i < b->rows_pool.size(); ++i)
+    if (b->m->lay->layers[i].own()) cudaFree(b->rows_pool[i]);
   cudaFree(b->d_table); cudaFree(b->d_seq); cudaFree(b->d_pos); cudaFree(b->d_next);
   cudaFree(b->d_part);
   delete b;
@@ -2048,6 +2048,7 @@ int b200_batch_add(b200_batch *b, int *seq) {
   for (int i = 0; i < b->max_seqs; ++i)
     if (b->len[i] < 0) {
       b->len[i] = 0;
+      b->first[i] = 0;
       *seq = i;
       return B200_OK;
     }
@@ -2058,7 +2059,7 @@ int b200_batch_remove(b200_batch *b, int seq) {
   if (!b || seq < 0 || seq >= b->max_seqs || b->len[seq] < 0)
     return fail(B200_EINVAL, "batch_remove: no such sequence");
   const int pages = (b->len[seq] + b->page - 1) / b->page;
-  for (int i = 0; i < pages; ++i)
+  for (int i = b->first[seq]; i < pages; ++i)
     b->free_pages.push_back(b->table[(size_t)seq * b->table_stride + i]);
   b->len[seq] = -1;
   return B200_OK;
@@ -2070,19 +2071,62 @@ int b200_batch_length(const b200_batch *b, int seq) {
 int b200_batch_free_pages(const b200_batch *b) { return b ? (int)b->free_pages.size() : 0; }
 float b200_batch_last_ms(const b200_batch *b) { return b ? b->last_ms : 0.f; }
 
+int b200_batch_step(b200_batch *b, int n_entries, const int *seqs, const int *counts, const int32_t *tokens, int n_want,
+                    const int32_t *want, float *logits_host, int32_t *next_tokens) {
+  if (!b || !seqs || !counts || !tokens || n_entries < 1 || n_entries > b->max_seqs || n_want < 0 || (n_want > 0 && !want))
+    return fail(B200_EINVAL, "batch_step: bad argument");
+  std::vector<char> seen((size_t)b->max_seqs, 0);
+  int64_t M = 0;
+  for (int i = 0; i < n_entries; ++i) {
+    const int s = seqs[i];
+    if (s < 0 || s >= b->max_seqs || b->len[s] < 0 || seen[(size_t)s])
+      return fail(B200_EINVAL, "batch_step: sequence %d is unknown or listed twice", s);
+    if (counts[i] < 1 || (int64_t)b->len[s] + counts[i] > b->max_context)
+      return fail(counts[i] < 1 ? B200_EINVAL : B200_ELIMIT, "batch_step: %d tokens for sequence %d at %d of %d positions", counts[i],
+                  s, b->len[s], b->max_context);
+    seen[(size_t)s] = 1;
+    M += counts[i];
+  }
+  if (M > (1 << 24))
+    return fail(B200_ELIMIT, "batch_step: %lld rows in one step", (long long)M);
+  for (int64_t r = 0; r < M; ++r)
+    if (tokens[r] < 0 || tokens[r] >= b->m->cfg.vocab)
+      return fail(B200_EINVAL, "batch_step: token %d at row %lld out of range", tokens[r], (long long)r);
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= M || (i > 0 && want[i] <= want[i - 1]))
+      return fail(B200_EINVAL, "batch_step: wanted rows must be ascending rows of the step");
+  for (int i = 0; i < n_entries; ++i)
+    if (int rc = batch_grow(b, seqs[i], counts[i])) {
+      // pages taken for this step go back: positions have not advanced
+      for (int k = 0; k < i; ++k)
+        batch_ungrow(b, seqs[k], counts[k]);
+      return rc;
+    }
+  std::vector<int32_t> rs((size_t)M), rp((size_t)M);
+  int64_t r = 0;
+  for (int i = 0; i < n_entries; ++i)
+    for (int k = 0; k < counts[i]; ++k, ++r) {
+      rs[(size_t)r] = seqs[i];
+      rp[(size_t)r] = b->len[seqs[i]] + k;
+    }
+  if (int rc = batch_rows(b, (int)M, tokens, rs.data(), rp.data(), n_want, want, logits_host, next_tokens)) {
+    for (int i = 0; i < n_entries; ++i)
+      batch_ungrow(b, seqs[i], counts[i]);
+    return rc;
+  }
+  for (int i = 0; i < n_entries; ++i) {
+    b->len[seqs[i]] += counts[i];
+    batch_release_passed(b, seqs[i]);
+  }
+  return B200_OK;
+}
+
 int b200_batch_prefill(b200_batch *b, int seq, const int32_t *tokens, int n, float *logits_host, int *next_token) {
-  if (!b || !tokens || n < 1 || seq < 0 || seq >= b->max_seqs || b->len[seq] < 0)
+  if (!b || !tokens || n < 1)
     return fail(B200_EINVAL, "batch_prefill: bad argument");
-  for (int i = 0; i < n; ++i)
-    if (tokens[i] < 0 || tokens[i] >= b->m->cfg.vocab)
-      return fail(B200_EINVAL, "batch_prefill: token %d at row %d out of range", tokens[i], i);
-  if (int rc = batch_grow(b, seq, n)) return rc;
-  std::vector<int32_t> rs((size_t)n, seq), rp((size_t)n);
-  for (int i = 0; i < n; ++i)
-    rp[(size_t)i] = b->len[seq] + i;
+  const int32_t last = n - 1;
   int32_t nxt = 0;
-  if (int rc = batch_rows(b, n, tokens, rs.data(), rp.data(), false, logits_host, &nxt)) return rc;
-  b->len[seq] += n;
+  if (int rc = b200_batch_step(b, 1, &seq, &n, tokens, 1, &last, logits_host, &nxt)) return rc;
   if (next_token) *next_token = nxt;
   return B200_OK;
 }
@@ -2091,26 +2135,11 @@ int b200_batch_decode(b200_batch *b, int n, const int *seqs, const int32_t *toke
                       int32_t *next_tokens) {
   if (!b || !seqs || !tokens || n < 1 || n > b->max_seqs)
     return fail(B200_EINVAL, "batch_decode: bad argument");
-  std::vector<int32_t> rs((size_t)n), rp((size_t)n);
-  std::vector<char> seen((size_t)b->max_seqs, 0);
-  for (int i = 0; i < n; ++i) {
-    const int s = seqs[i];
-    if (s < 0 || s >= b->max_seqs || b->len[s] < 0 || seen[(size_t)s])
-      return fail(B200_EINVAL, "batch_decode: sequence %d is unknown or listed twice", s);
-    if (tokens[i] < 0 || tokens[i] >= b->m->cfg.vocab)
-      return fail(B200_EINVAL, "batch_decode: token %d of sequence %d out of range", tokens[i], s);
-    seen[(size_t)s] = 1;
-  }
+  std::vector<int32_t> all((size_t)n);
+  std::vector<int> ones((size_t)n, 1);
   for (int i = 0; i < n; ++i)
-    if (int rc = batch_grow(b, seqs[i], 1)) return rc;
-  for (int i = 0; i < n; ++i) {
-    rs[(size_t)i] = seqs[i];
-    rp[(size_t)i] = b->len[seqs[i]];
-  }
-  if (int rc = batch_rows(b, n, tokens, rs.data(), rp.data(), true, logits_host, next_tokens)) return rc;
-  for (int i = 0; i < n; ++i)
-    b->len[seqs[i]] += 1;
-  return B200_OK;
+    all[(size_t)i] = i;
+  return b200_batch_step(b, n, seqs, ones.data(), tokens, n, all.data(), logits_host, next_tokens);
 }
 
 int b200_model_read_new_kv_rows(b200_model *m, float *host) {
@@ -2164,6 +2193,7 @@ int b200_model_read_trace(b200_model *m, long long *host, int64_t capacity) {
 
 int64_t b200_model_step_bytes(const b200_model *m, int ctx) {
   if (!m) return 0;
+  if (m->lay) return layered_step_bytes(m, ctx);
   const b200_model_config &c = m->cfg;
   int64_t b = 0;
   for (const auto &L : m->layers) {

@@ -42,11 +42,9 @@
 // an error, all roles fall through, tensor memory is released and the host
 // call fails.
 #include "common.cuh"
-
-#include <cuda.h>
+#include "tc.cuh"
 
 #include <algorithm>
-#include <mutex>
 
 namespace b200 {
 
@@ -58,8 +56,6 @@ constexpr int kMaxStages = 8;
 // weights arrive as bf16)
 constexpr int kThreadsConv = 320, kThreadsPre = 320;
 constexpr int kMaxPartialTiles = 320;          // split-K: 128 x 128 f32 partial tiles in the workspace
-constexpr uint32_t kSpin = 1u << 26;
-constexpr unsigned long long kWaitNs = 2000000000ull;
 
 // Shared-memory stage for a k block of BKT elements (64: 128-byte swizzle rows, 32: 64-byte rows).
 // PRE: the weight tile is loaded as bf16 (converted by a pass over the weights before the
@@ -81,66 +77,6 @@ struct Bars {
   int abort_flag;
 };
 
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ unsigned long long now_ns() {
-  unsigned long long t;
-  asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
-  return t;
-}
-__device__ __forceinline__ void mbar_init(uint64_t *bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count));
-}
-__device__ __forceinline__ void mbar_expect_tx(uint64_t *bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint64_t *bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ bool mbar_try(uint64_t *bar, uint32_t parity) {
-  uint32_t ok;
-  asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}"
-               : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-  return ok != 0;
-}
-// Bounded wait; false when it gave up or the CTA already failed.
-__device__ __forceinline__ bool mbar_wait(uint64_t *bar, uint32_t parity, volatile int *ab, int *err, int code) {
-  unsigned long long t0 = 0;
-  for (uint32_t it = 0; it < kSpin; ++it) {
-    if (mbar_try(bar, parity))
-      return !*ab;
-    if ((it & 0x3FF) == 0x3FF) {
-      if (*ab)
-        return false;
-      const unsigned long long t = now_ns();
-      if (t0 == 0)
-        t0 = t;
-      else if (t - t0 > kWaitNs)
-        break;
-    }
-  }
-  atomicCAS(err, 0, code);
-  *ab = 1;
-  return false;
-}
-__device__ __forceinline__ void tma_load_2d(void *dst, const CUtensorMap *map, int x, int y, uint64_t *bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-      ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y)
-      : "memory");
-}
-// K-major operand tile in shared memory, rows of 128 bytes (128-byte swizzle) or
-// 64 bytes (64-byte swizzle): start address / 16, leading byte offset (unused for
-// swizzled K-major: 1), stride byte offset = 8 rows, descriptor version 1,
-// layout 2 (128-byte swizzle) or 4 (64-byte swizzle).
-template <int BKT> __device__ __forceinline__ uint64_t smem_desc(uint32_t addr) {
-  uint64_t d = 0;
-  d |= (uint64_t)((addr & 0x3FFFFu) >> 4);
-  d |= (uint64_t)1 << 16;
-  d |= (uint64_t)((8 * BKT * 2) >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)(BKT == 64 ? 2 : 4) << 61;
-  return d;
-}
 // kind::f16 instruction descriptor: D = f32, A = B = bf16, both K-major, N = 128, M = 128.
 template <int BNT> struct Idesc {
   static constexpr uint32_t value =
@@ -155,10 +91,6 @@ __device__ __forceinline__ void mma_bf16(uint32_t tmem_d, uint64_t da, uint64_t 
       ::"r"(tmem_d), "l"(da), "l"(db), "r"(Idesc<BNT>::value), "r"(accumulate)
       : "memory");
 }
-__device__ __forceinline__ void tc_commit(uint64_t *bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-
 struct GemmParams {
   int M, N, K;                 // N = weight rows covered by this launch; K = packed k (multiple of 64)
   int n_off;                   // first weight row of the launch: scale, bias, residual and C are indexed n_off + n
@@ -864,39 +796,6 @@ split_activations_warp_kernel(const float *A, int64_t lda, int M, int K, const f
     hrow[pos >> 2] = make_uint2(hb[0] | (hb[1] << 16), hb[2] | (hb[3] << 16));
     lrow[pos >> 2] = make_uint2(lb[0] | (lb[1] << 16), lb[2] | (lb[3] << 16));
   }
-}
-
-using EncodeFn = CUresult (*)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
-                              const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
-                              CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeFn encode_fn() {
-  static EncodeFn fn = nullptr;
-  static std::once_flag once;
-  std::call_once(once, [] {
-    void *p = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeFn>(p);
-  });
-  return fn;
-}
-
-int make_map(CUtensorMap *map, CUtensorMapDataType dt, int bk, void *base, uint64_t inner, uint64_t rows,
-             uint64_t pitch_bytes, CUtensorMapSwizzle swz, int box_rows = 128) {
-  EncodeFn fn = encode_fn();
-  if (!fn)
-    return fail(B200_ECUDA, "gemm_w8: cuTensorMapEncodeTiled is not available from this driver");
-  const cuuint64_t dims[2] = {inner, rows};
-  const cuuint64_t strides[1] = {pitch_bytes};
-  const cuuint32_t box[2] = {(cuuint32_t)bk, (cuuint32_t)box_rows};
-  const cuuint32_t estr[2] = {1, 1};
-  const CUresult rc = fn(map, dt, 2, base, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, swz,
-                         CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (rc != CUDA_SUCCESS)
-    return fail(B200_ECUDA, "gemm_w8: cuTensorMapEncodeTiled failed (%d)", (int)rc);
-  return B200_OK;
 }
 
 } // namespace

@@ -1,0 +1,470 @@
+// Models of described layers: creation, loading by tensor name, and the step over M rows of any
+// mix of sequences.  The session's decode step (captured into a CUDA graph), its prefill and the
+// batch calls of engine.cu all come through layered_rows / layered_issue_step; what differs is
+// where a row's cache lines are (CacheView): the session's contiguous cache is one page.
+//
+// A layer x += mixer(h) + ff(h), h = RMSNorm(x), runs as
+//   in    one contraction of the normalised row with every matrix that reads it: queries, latent
+//         and key part, router logits, and the (gate, up) pairs of a dense feed-forward (gated in
+//         the epilogue)
+//   latent attention over the cache (latent.cu)
+//   out   one contraction of [attention | gated feed-forward] with [W_o | W_down], added to x
+// or, with experts, their own two contractions (gemv_rows.cu, experts.cu).
+#include "engine.cuh"
+
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+
+namespace b200 {
+
+namespace {
+
+// src rows [rows][cols] (row-major, tight) -> dst row (row0 + r * step), columns col0..
+template <typename S, typename D>
+__global__ void place_rows_kernel(const S *src, int cols, D *dst, int64_t ld, int64_t row0, int64_t step, int64_t col0) {
+  const int64_t r = blockIdx.x;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x)
+    dst[(row0 + r * step) * ld + col0 + c] = from_float<D>(to_float(src[r * cols + c]));
+}
+
+template <typename T>
+__global__ void embed_table_kernel(const T *table, int64_t ld, const int32_t *tokens, float *x, int H) {
+  const T *src = table + (int64_t)tokens[blockIdx.x] * ld;
+  for (int i = threadIdx.x; i < H; i += blockDim.x)
+    x[(int64_t)blockIdx.x * H + i] = to_float(src[i]);
+}
+
+__global__ void gather_rows_kernel(const float *x, const int32_t *rows, float *y, int H) {
+  const float *src = x + (int64_t)rows[blockIdx.x] * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x)
+    y[(int64_t)blockIdx.x * H + i] = src[i];
+}
+
+int64_t pad_to(int64_t n, int64_t a) { return (n + a - 1) / a * a; }
+
+int own_alloc(std::vector<void *> &owned, void **p, size_t bytes) {
+  if (int rc = dev_alloc(p, bytes)) return rc;
+  owned.push_back(*p);
+  B200_CUDA(cudaMemset(*p, 0, bytes ? bytes : 16));
+  return B200_OK;
+}
+template <typename T> int own_array(std::vector<void *> &owned, T **p, int64_t n) {
+  return own_alloc(owned, (void **)p, (size_t)(n > 0 ? n : 1) * sizeof(T));
+}
+size_t elem(int dtype) { return dtype == B200_F32 ? 4 : 2; }
+
+void release(std::vector<void *> &owned) {
+  for (void *p : owned)
+    cudaFree(p);
+  owned.clear();
+}
+
+int make_matrix(LayeredState *s, RowMatrix *w, int64_t N, int64_t K) {
+  w->N = (int)N;
+  w->K = (int)K;
+  w->ld = pad_to(K, 8);
+  return own_alloc(s->owned, &w->w, (size_t)N * w->ld * elem(s->dtype));
+}
+
+void add_rows(LayeredState *s, const std::string &name, const RowMatrix &w, int rows, int cols, int64_t row0,
+              int64_t step = 1, int64_t col0 = 0) {
+  s->tensors[name] = LayeredTensor{rows, cols, s->dtype, w.w, w.ld, row0, step, col0, false};
+}
+int add_vector(LayeredState *s, const std::string &name, float **p, int n) {
+  if (int rc = own_array(s->owned, p, n)) return rc;
+  s->tensors[name] = LayeredTensor{1, n, B200_F32, *p, n, 0, 1, 0, false};
+  return B200_OK;
+}
+
+int check_layer(const b200_layer_config &c, int i, const b200_layer_config *all) {
+  if (c.mixer != B200_MIX_LATENT)
+    return fail(B200_EINVAL, "create_layered: layer %d has an unknown mixer %d", i, c.mixer);
+  LatentDims d{};
+  d.heads = c.heads; d.dim = c.dim; d.rot = c.rot_dim; d.vdim = c.vdim; d.rank = c.kv_rank;
+  if (int rc = latent_limits(d)) return rc;
+  if (c.window < 0 || !std::isfinite(c.scale) || !(c.rot_base > 0.f))
+    return fail(B200_EINVAL, "create_layered: layer %d: bad window, scale or rotation base", i);
+  if (c.kv_from >= 0) {
+    if (c.kv_from >= i || all[c.kv_from].kv_from >= 0)
+      return fail(B200_EINVAL, "create_layered: layer %d takes the cache of layer %d, which has none of its own before it", i, c.kv_from);
+    const b200_layer_config &o = all[c.kv_from];
+    if (o.kv_rank != c.kv_rank || o.rot_dim != c.rot_dim || o.rot_base != c.rot_base)
+      return fail(B200_EINVAL, "create_layered: layer %d and the layer whose cache it takes differ in latent or rotation", i);
+  }
+  if (c.ff_kind != B200_FF_NONE && c.ff_kind != B200_FF_GATED && c.ff_kind != B200_FF_EXPERTS)
+    return fail(B200_EINVAL, "create_layered: layer %d has an unknown feed-forward %d", i, c.ff_kind);
+  if (c.ff_kind != B200_FF_NONE && (c.ff < 1 || !(c.limit > 0.f)))
+    return fail(B200_EINVAL, "create_layered: layer %d: bad feed-forward", i);
+  if (c.ff_kind == B200_FF_EXPERTS && (c.experts < 1 || c.top < 1 || c.top > c.experts || c.experts > 1024))
+    return fail(B200_EINVAL, "create_layered: layer %d: %d of %d experts", i, c.top, c.experts);
+  return B200_OK;
+}
+
+int build_layer(LayeredState *s, LayeredLayer &L, int i, int W) {
+  const b200_layer_config &c = L.cfg;
+  LatentDims &d = L.d;
+  d.heads = c.heads; d.dim = c.dim; d.rot = c.rot_dim; d.vdim = c.vdim; d.rank = c.kv_rank;
+  d.window = c.window;
+  d.scale = c.scale;
+  d.row = pad_to(d.rank + d.rot, 8);
+  L.source = c.kv_from >= 0 ? c.kv_from : i;
+  L.att = d.heads * d.vdim;
+  L.gate = Gate{c.limit, c.gate_slope, c.up_offset};
+  const bool dense = c.ff_kind == B200_FF_GATED, experts = c.ff_kind == B200_FF_EXPERTS;
+  const int nq = d.heads * (d.dim + d.rot);
+  int n = nq;
+  L.off_down = n;
+  if (L.own()) n += d.rank + d.rot;
+  L.off_router = n;
+  if (experts) n += c.experts;
+  L.plain = (int)pad_to(n, 4);
+  const std::string p = "l" + std::to_string(i) + ".";
+  if (int rc = make_matrix(s, &L.in, L.plain + (dense ? 2 * c.ff : 0), W)) return rc;
+  add_rows(s, p + "mix.q", L.in, nq, W, 0);
+  if (L.own()) add_rows(s, p + "mix.dkv", L.in, d.rank + d.rot, W, L.off_down);
+  if (experts) add_rows(s, p + "mlp.router", L.in, c.experts, W, L.off_router);
+  if (int rc = make_matrix(s, &L.ukv, (int64_t)d.heads * (d.dim + d.vdim), d.rank)) return rc;
+  L.uk = L.uv = L.ukv;
+  L.uk.N = d.heads * d.dim;
+  L.uv.N = L.att;
+  L.uv.w = (char *)L.ukv.w + (size_t)L.uk.N * L.ukv.ld * elem(s->dtype);
+  add_rows(s, p + "mix.uk", L.uk, L.uk.N, d.rank, 0);
+  add_rows(s, p + "mix.uv", L.uv, L.uv.N, d.rank, 0);
+  if (int rc = make_matrix(s, &L.out, W, L.att + (dense ? c.ff : 0))) return rc;
+  add_rows(s, p + "mix.o", L.out, W, L.att, 0);
+  if (dense) {
+    add_rows(s, p + "mlp.gate", L.in, c.ff, W, L.plain, 2);
+    add_rows(s, p + "mlp.up", L.in, c.ff, W, L.plain + 1, 2);
+    add_rows(s, p + "mlp.down", L.out, W, c.ff, 0, 1, L.att);
+  }
+  if (experts) {
+    if (int rc = make_matrix(s, &L.expert_in, (int64_t)c.experts * 2 * c.ff, W)) return rc;
+    if (int rc = make_matrix(s, &L.expert_out, (int64_t)c.experts * W, c.ff)) return rc;
+    for (int e = 0; e < c.experts; ++e) {
+      const std::string q = p + "mlp.e" + std::to_string(e) + ".";
+      add_rows(s, q + "gate", L.expert_in, c.ff, W, (int64_t)e * 2 * c.ff, 2);
+      add_rows(s, q + "up", L.expert_in, c.ff, W, (int64_t)e * 2 * c.ff + 1, 2);
+      add_rows(s, q + "down", L.expert_out, W, c.ff, (int64_t)e * W);
+    }
+  }
+  if (int rc = add_vector(s, p + "norm1", &L.norm, W)) return rc;
+  if (L.own())
+    if (int rc = add_vector(s, p + "mix.dkv.norm", &L.down_norm, d.rank)) return rc;
+  std::vector<float> f((size_t)std::max(1, d.rot / 2));
+  for (int k = 0; k < d.rot / 2; ++k)
+    f[(size_t)k] = (float)std::pow((double)c.rot_base, -2.0 * k / d.rot);
+  if (int rc = own_array(s->owned, &L.inv_freq, (int64_t)f.size())) return rc;
+  B200_CUDA(cudaMemcpy(L.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice));
+  s->ldp = std::max(s->ldp, (int)pad_to(L.plain, 4));
+  s->ldc = std::max(s->ldc, (int)L.out.ld);
+  s->ldq = std::max(s->ldq, d.heads * (d.rank + d.rot));
+  if (experts) {
+    s->max_mid = std::max(s->max_mid, c.top * c.ff);
+    s->max_top = std::max(s->max_top, c.top);
+    s->max_ff = std::max(s->max_ff, c.ff);
+    s->max_experts = std::max(s->max_experts, c.experts);
+  }
+  return B200_OK;
+}
+
+// Activations for up to `rows` rows, contexts up to `ctx` positions.
+int reserve(b200_model *m, LayeredWs &ws, int rows, int ctx) {
+  LayeredState *s = m->lay;
+  if (rows <= ws.rows && ctx <= ws.ctx)
+    return B200_OK;
+  rows = std::max(rows, ws.rows);
+  ctx = std::max(ctx, ws.ctx);
+  B200_CUDA(cudaStreamSynchronize(m->stream));
+  release(ws.owned);
+  ws = LayeredWs();
+  const int W = m->cfg.hidden;
+  int64_t part = 0;
+  for (const LayeredLayer &L : s->layers)
+    for (int r = 1; r <= rows; r = r < 512 || r == rows ? r + 1 : rows)   // beyond 512 rows there is one share
+      part = std::max(part, latent_scratch_floats(L.d, r, latent_splits(L.d, r, ctx)));
+  auto &o = ws.owned;
+  int rc = own_array(o, &ws.x, (int64_t)rows * W);
+  if (!rc) rc = own_array(o, &ws.proj, (int64_t)rows * s->ldp);
+  if (!rc) rc = own_array(o, &ws.qabs, (int64_t)rows * s->ldq);
+  if (!rc) rc = own_array(o, &ws.part, part);
+  if (!rc) rc = own_array(o, &ws.cat, (int64_t)rows * s->ldc);
+  if (!rc) rc = own_array(o, &ws.mid, (int64_t)rows * s->max_mid);
+  if (!rc) rc = own_array(o, &ws.weight, (int64_t)rows * s->max_top);
+  if (!rc) rc = own_array(o, &ws.ids, (int64_t)rows * s->max_top);
+  if (!rc) rc = own_array(o, &ws.row_seq, rows);
+  if (!rc) rc = own_array(o, &ws.row_pos, rows);
+  if (!rc) rc = own_array(o, &ws.tokens, rows);
+  if (rc) {
+    release(ws.owned);
+    ws = LayeredWs();
+    return rc;
+  }
+  ws.rows = rows;
+  ws.ctx = ctx;
+  return B200_OK;
+}
+
+// All layers over M rows, GEMV-shaped (few rows, or 32-bit).
+int row_layers(b200_model *m, LayeredWs &ws, float *x, int M, const CacheView &cv, void *const *pools, int max_ctx,
+               cudaStream_t st) {
+  LayeredState *s = m->lay;
+  const int W = m->cfg.hidden;
+  const float eps = m->cfg.eps;
+  for (LayeredLayer &L : s->layers) {
+    const b200_layer_config &c = L.cfg;
+    if (int rc = gemv_rows_launch(s->dtype, L.in, x, W, M, L.norm, eps, ws.proj, s->ldp, false, L.plain, ws.cat + L.att,
+                                  s->ldc, L.gate, st))
+      return rc;
+    void *pool = pools[L.source];
+    if (int rc = latent_prep_launch(s->dtype, L.d, ws.proj, s->ldp, M, L.uk, L.inv_freq, ws.qabs, L.own(), L.off_down,
+                                    L.down_norm, eps, pool, cv, st))
+      return rc;
+    const int splits = latent_splits(L.d, M, max_ctx);
+    if (int rc = latent_attend_launch(s->dtype, L.d, ws.qabs, M, pool, cv, splits, max_ctx, ws.part, st)) return rc;
+    if (int rc = latent_value_launch(s->dtype, L.d, ws.part, M, splits, L.uv, ws.cat, s->ldc, false, st)) return rc;
+    if (c.ff_kind == B200_FF_EXPERTS) {
+      if (int rc = expert_rows_launch(s->dtype, L.expert_in, L.expert_out, c.ff, c.experts, c.top, L.gate, x, W, M,
+                                      L.norm, eps, ws.proj + L.off_router, s->ldp, &L.out, ws.cat, s->ldc, ws.mid,
+                                      ws.ids, ws.weight, st))
+        return rc;
+    } else if (int rc = gemv_rows_launch(s->dtype, L.out, ws.cat, s->ldc, M, nullptr, 0.f, x, W, true, W, nullptr, 0,
+                                         L.gate, st)) {
+      return rc;
+    }
+  }
+  return B200_OK;
+}
+
+int embed_tokens(b200_model *m, const int32_t *tokens, float *x, int M, cudaStream_t st) {
+  LayeredState *s = m->lay;
+  const int W = m->cfg.hidden;
+  if (s->dtype == B200_F32)
+    embed_table_kernel<float><<<M, 128, 0, st>>>((const float *)s->embed.w, s->embed.ld, tokens, x, W);
+  else
+    embed_table_kernel<bf16><<<M, 128, 0, st>>>((const bf16 *)s->embed.w, s->embed.ld, tokens, x, W);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+int head(b200_model *m, const float *x, int n, float *logits, cudaStream_t st) {
+  LayeredState *s = m->lay;
+  return gemv_rows_launch(s->dtype, s->embed, x, m->cfg.hidden, n, s->final_norm, m->cfg.eps, logits, m->cfg.vocab, false,
+                          m->cfg.vocab, nullptr, 0, Gate{}, st);
+}
+
+} // namespace
+
+int layered_ready(b200_model *m) {
+  for (const auto &t : m->lay->tensors)
+    if (!t.second.set)
+      return fail(B200_ESTATE, "finalize: tensor %s is missing", t.first.c_str());
+  return B200_OK;
+}
+
+void layered_destroy(b200_model *m) {
+  LayeredState *s = m->lay;
+  if (!s) return;
+  release(s->one.owned);
+  release(s->many.owned);
+  release(s->owned);
+  cudaFree(s->x_want); cudaFree(s->h_want); cudaFree(s->logits); cudaFree(s->want); cudaFree(s->next);
+  cudaFree(s->gemm_ws);
+  delete s;
+  m->lay = nullptr;
+}
+
+int layered_clear_cache(b200_model *m) {
+  LayeredState *s = m->lay;
+  for (LayeredLayer &L : s->layers)
+    if (L.cache)
+      B200_CUDA(cudaMemsetAsync(L.cache, 0, (size_t)m->cfg.max_len * L.d.row * elem(s->dtype), m->stream));
+  return B200_OK;
+}
+
+int layered_issue_step(b200_model *m, cudaStream_t st) {
+  LayeredState *s = m->lay;
+  if (int rc = reserve(m, s->one, 1, m->cfg.max_len)) return rc;
+  std::vector<void *> pools;
+  for (LayeredLayer &L : s->layers)
+    pools.push_back(L.cache);
+  const CacheView cv{s->zero, m->d_state + 1, s->zero, 1, m->cfg.max_len};
+  if (int rc = embed_tokens(m, m->d_state, m->x, 1, st)) return rc;
+  if (int rc = row_layers(m, s->one, m->x, 1, cv, pools.data(), m->cfg.max_len, st)) return rc;
+  return head(m, m->x, 1, m->logits, st);
+}
+
+// M rows (host arrays) of any sequences, in chunks of rows; the logits of the `want` rows.
+int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row_seq, const int32_t *row_pos,
+                 const int32_t *table_dev, int table_stride, int page, void *const *pools, int max_ctx, int n_want,
+                 const int32_t *want, float *logits_host, int32_t *next_host) {
+  LayeredState *s = m->lay;
+  const int W = m->cfg.hidden;
+  cudaStream_t st = m->stream;
+  const int chunk = s->dtype == B200_F32 ? 512 : 4096;
+  if (int rc = reserve(m, s->many, std::min(M, chunk), max_ctx)) return rc;
+  if (n_want > s->want_cap) {
+    B200_CUDA(cudaStreamSynchronize(st));
+    cudaFree(s->x_want); cudaFree(s->h_want); cudaFree(s->logits); cudaFree(s->want); cudaFree(s->next);
+    s->x_want = s->logits = nullptr;
+    s->h_want = nullptr;
+    s->want = s->next = nullptr;
+    s->want_cap = 0;
+    if (int rc = dev_alloc((void **)&s->x_want, (size_t)n_want * W * 4)) return rc;
+    if (int rc = dev_alloc((void **)&s->h_want, (size_t)n_want * pad_to(W, 8) * 2)) return rc;
+    if (int rc = dev_alloc((void **)&s->logits, (size_t)n_want * m->cfg.vocab * 4)) return rc;
+    if (int rc = dev_alloc((void **)&s->want, (size_t)n_want * 4)) return rc;
+    if (int rc = dev_alloc((void **)&s->next, (size_t)n_want * 4)) return rc;
+    s->want_cap = n_want;
+  }
+  LayeredWs &ws = s->many;
+  std::vector<int32_t> local;
+  int done = 0;                          // wanted rows gathered so far
+  for (int m0 = 0; m0 < M; m0 += chunk) {
+    const int n = std::min(chunk, M - m0);
+    B200_CUDA(cudaMemcpyAsync(ws.tokens, tokens + m0, (size_t)n * 4, cudaMemcpyHostToDevice, st));
+    B200_CUDA(cudaMemcpyAsync(ws.row_seq, row_seq + m0, (size_t)n * 4, cudaMemcpyHostToDevice, st));
+    B200_CUDA(cudaMemcpyAsync(ws.row_pos, row_pos + m0, (size_t)n * 4, cudaMemcpyHostToDevice, st));
+    const CacheView cv{ws.row_seq, ws.row_pos, table_dev, table_stride, page};
+    if (int rc = embed_tokens(m, ws.tokens, ws.x, n, st)) return rc;
+    if (int rc = row_layers(m, ws, ws.x, n, cv, pools, max_ctx, st)) return rc;
+    local.clear();
+    for (int k = done; k < n_want && want[k] < m0 + n; ++k)
+      local.push_back(want[k] - m0);
+    if (!local.empty()) {
+      B200_CUDA(cudaMemcpyAsync(s->want, local.data(), local.size() * 4, cudaMemcpyHostToDevice, st));
+      gather_rows_kernel<<<(unsigned)local.size(), 128, 0, st>>>(ws.x, s->want, s->x_want + (int64_t)done * W, W);
+      B200_LAUNCH_CHECK();
+      done += (int)local.size();
+      B200_CUDA(cudaStreamSynchronize(st));   // `local` is reused
+    }
+  }
+  if (n_want > 0) {
+    if (int rc = head(m, s->x_want, n_want, s->logits, st)) return rc;
+    if (int rc = argmax_rows_launch(s->logits, m->cfg.vocab, n_want, s->next, st)) return rc;
+    if (logits_host)
+      B200_CUDA(cudaMemcpyAsync(logits_host, s->logits, (size_t)n_want * m->cfg.vocab * 4, cudaMemcpyDeviceToHost, st));
+    if (next_host)
+      B200_CUDA(cudaMemcpyAsync(next_host, s->next, (size_t)n_want * 4, cudaMemcpyDeviceToHost, st));
+  }
+  return B200_OK;
+}
+
+int64_t layered_step_bytes(const b200_model *m, int ctx) {
+  const LayeredState *s = m->lay;
+  const int64_t e = (int64_t)elem(s->dtype), W = m->cfg.hidden;
+  auto mat = [&](const RowMatrix &w) { return (int64_t)w.N * w.K * e; };
+  int64_t b = (int64_t)m->cfg.vocab * W * e + W * e + W * 4;   // head, embedding row, final norm
+  for (const LayeredLayer &L : s->layers) {
+    b += mat(L.in) + mat(L.out) + mat(L.ukv) + W * 4;
+    if (L.cfg.ff_kind == B200_FF_EXPERTS)   // the chosen experts only
+      b += (mat(L.expert_in) + mat(L.expert_out)) / L.cfg.experts * L.cfg.top;
+    const int64_t seen = L.d.window > 0 ? std::min(L.d.window, ctx + 1) : ctx + 1;
+    b += seen * (L.d.rank + L.d.rot) * e;
+  }
+  return b;
+}
+
+} // namespace b200
+
+using namespace b200;
+
+extern "C" {
+
+int b200_model_create_layered(const b200_model_config *cfg, const b200_layer_config *layers, int dtype, b200_model **out) {
+  if (!cfg || !layers || !out)
+    return fail(B200_EINVAL, "create_layered: null argument");
+  if (dtype != B200_F32 && dtype != B200_BF16)
+    return fail(B200_EINVAL, "create_layered: dtype must be B200_F32 or B200_BF16");
+  if (cfg->hidden < 1 || cfg->n_layers < 1 || cfg->vocab < 1 || cfg->max_len < 1 || !(cfg->eps >= 0.f))
+    return fail(B200_EINVAL, "create_layered: bad architecture");
+  if (cfg->tp_size > 1)
+    return fail(B200_EINVAL, "create_layered: single-GPU sessions only");
+  for (int i = 0; i < cfg->n_layers; ++i)
+    if (int rc = check_layer(layers[i], i, layers)) return rc;
+  b200_model_config base{};
+  base.hidden = cfg->hidden; base.n_layers = cfg->n_layers; base.vocab = cfg->vocab; base.max_len = cfg->max_len;
+  base.eps = cfg->eps; base.head_dim = 64; base.tp_size = 1;
+  b200_model *m = nullptr;
+  if (int rc = model_allocate(base, &m)) return rc;
+  LayeredState *s = new LayeredState();
+  m->lay = s;
+  s->dtype = dtype;
+  s->layers.resize(cfg->n_layers);
+  int rc = make_matrix(s, &s->embed, cfg->vocab, cfg->hidden);
+  if (!rc) {
+    add_rows(s, "embed", s->embed, cfg->vocab, cfg->hidden, 0);
+    rc = add_vector(s, "final.norm", &s->final_norm, cfg->hidden);
+  }
+  if (!rc) rc = own_array(s->owned, &s->zero, 4);
+  bool all = false;
+  for (int i = 0; i < cfg->n_layers && !rc; ++i) {
+    LayeredLayer &L = s->layers[i];
+    L.cfg = layers[i];
+    rc = build_layer(s, L, i, cfg->hidden);
+    all = all || L.cfg.window == 0;
+    s->window = std::max(s->window, L.cfg.window);
+    if (!rc && L.own())
+      rc = own_alloc(s->owned, &L.cache, (size_t)cfg->max_len * L.d.row * elem(dtype));
+  }
+  if (all)
+    s->window = 0;
+  for (LayeredLayer &L : s->layers)
+    L.cache = s->layers[L.source].cache;
+  if (rc) {
+    b200_model_destroy(m);
+    return rc;
+  }
+  *out = m;
+  return B200_OK;
+}
+
+int b200_model_set_tensor(b200_model *m, const char *name, int dtype, const void *host, int64_t rows, int64_t cols) {
+  if (!m || !name || !host || !m->lay)
+    return fail(B200_EINVAL, "set_tensor: a model of described layers, a name and data are required");
+  if (m->finalized)
+    return fail(B200_ESTATE, "set_tensor: model already finalised");
+  if (dtype != B200_F32 && dtype != B200_BF16)
+    return fail(B200_EINVAL, "set_tensor: %s: dtype must be B200_F32 or B200_BF16", name);
+  auto it = m->lay->tensors.find(name);
+  if (it == m->lay->tensors.end())
+    return fail(B200_EINVAL, "set_tensor: the model has no tensor %s", name);
+  LayeredTensor &t = it->second;
+  if (rows != t.rows || cols != t.cols)
+    return fail(B200_EINVAL, "set_tensor: %s is [%d, %d], got [%lld, %lld]", name, t.rows, t.cols, (long long)rows, (long long)cols);
+  const size_t bytes = (size_t)rows * cols * elem(dtype);
+  void *d = nullptr;
+  if (int rc = dev_alloc(&d, bytes)) return rc;
+  cudaStream_t st = m->stream;
+  int rc = B200_OK;
+  if (cudaMemcpyAsync(d, host, bytes, cudaMemcpyHostToDevice, st) != cudaSuccess)
+    rc = fail(B200_ECUDA, "set_tensor: upload failed");
+  if (!rc) {
+    const unsigned g = (unsigned)rows;
+    if (dtype == B200_F32 && t.dtype == B200_F32)
+      place_rows_kernel<float, float><<<g, 256, 0, st>>>((const float *)d, (int)cols, (float *)t.dst, t.ld, t.row0, t.step, t.col0);
+    else if (dtype == B200_F32)
+      place_rows_kernel<float, bf16><<<g, 256, 0, st>>>((const float *)d, (int)cols, (bf16 *)t.dst, t.ld, t.row0, t.step, t.col0);
+    else if (t.dtype == B200_F32)
+      place_rows_kernel<bf16, float><<<g, 256, 0, st>>>((const bf16 *)d, (int)cols, (float *)t.dst, t.ld, t.row0, t.step, t.col0);
+    else
+      place_rows_kernel<bf16, bf16><<<g, 256, 0, st>>>((const bf16 *)d, (int)cols, (bf16 *)t.dst, t.ld, t.row0, t.step, t.col0);
+    count_launch();
+    if (cudaGetLastError() != cudaSuccess || cudaStreamSynchronize(st) != cudaSuccess)
+      rc = fail(B200_ECUDA, "set_tensor: %s: placing the rows failed", name);
+  }
+  cudaFree(d);
+  if (!rc)
+    t.set = true;
+  return rc;
+}
+
+int b200_model_read_residual(b200_model *m, float *host, int n) {
+  if (!m || !host || !m->lay || n < 1 || n > m->lay->many.rows)
+    return fail(B200_EINVAL, "read_residual: bad argument");
+  B200_CUDA(cudaMemcpyAsync(host, m->lay->many.x, (size_t)n * m->cfg.hidden * 4, cudaMemcpyDeviceToHost, m->stream));
+  B200_CUDA(cudaStreamSynchronize(m->stream));
+  return B200_OK;
+}
+
+} // extern "C"

@@ -13,8 +13,7 @@ import time
 
 import numpy as np
 
-from . import _lib
-from .config import ModelConfig
+from . import _lib, safetensors_file
 from .synthetic import tensor_list
 
 _SLOT = {"q": _lib.T_Q, "k": _lib.T_K, "v": _lib.T_V, "o": _lib.T_O,
@@ -34,12 +33,14 @@ def greedy_sample(logits: np.ndarray) -> int:
 
 
 class ModelSession:
-    def __init__(self, cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1):
+    """A single-sequence session.  cfg: ModelConfig, or LayeredConfig for a model of described
+    layers (loaded by load_safetensors / load_named)."""
+
+    def __init__(self, cfg, tp_rank: int = 0, tp_size: int = 1):
         self.cfg = cfg
         self.lib = _lib.load()
         self._h = C.c_void_p()
-        self._cfg_c = cfg.to_c(tp_rank, tp_size)
-        _lib.check(self.lib.b200_model_create(C.byref(self._cfg_c), C.byref(self._h)))
+        _lib.check(cfg.create(self.lib, self._h, tp_rank, tp_size))
         self.position_ = 0
         self._logits = np.zeros(cfg.vocab, dtype=np.float32)
         self.tp_rank, self.tp_size = tp_rank, tp_size
@@ -117,6 +118,27 @@ class ModelSession:
         if save_packed is not None:
             _lib.check(self.lib.b200_model_save_packed(self._h, str(save_packed).encode()))
         self.finalize()
+
+    def load_named(self, tensors):
+        """Tensors by name for a model of described layers, {name: [out, in] array}: float32, or
+        uint16 holding bfloat16 patterns."""
+        for name, a in tensors.items():
+            a = np.asarray(a)
+            bf16 = a.dtype == np.uint16
+            a = np.ascontiguousarray(a, dtype=np.uint16 if bf16 else np.float32)
+            rows, cols = a.shape if a.ndim == 2 else (1, a.size)
+            _lib.check(self.lib.b200_model_set_tensor(self._h, name.encode(), _lib.BF16 if bf16 else _lib.F32,
+                                                      a.ctypes.data, rows, cols))
+        self.finalize()
+
+    def load_safetensors(self, path):
+        """load_named from a safetensors file."""
+        tensors = {}
+        for name, (dtype, a) in safetensors_file.read(path).items():
+            if dtype not in ("BF16", "F32", "F16"):
+                raise ValueError(f"{path}: tensor {name} of type {dtype}")
+            tensors[name] = a
+        self.load_named(tensors)
 
     def set_linear_quantised(self, layer, name, kind, w, scale, scale_dtype, signed, K, N, group=0):
         w = np.ascontiguousarray(w)
@@ -306,6 +328,29 @@ class BatchSession:
         _lib.check(self.lib.b200_batch_decode(self._h, n, sq.ctypes.data, tk.ctypes.data,
                                               out.ctypes.data if want_logits else None, nxt.ctypes.data))
         return out, nxt
+
+    def step(self, entries, want=None, want_logits=True):
+        """One mixed step: entries [(seq, next tokens)], want: per entry the places among its tokens
+        whose logits are asked for (default: the last).  Returns (logits [n, vocab] or None, first
+        maxima [n]), in the order of entries and places."""
+        if want is None:
+            want = [[len(t) - 1] for _, t in entries]
+        seqs = np.ascontiguousarray([s for s, _ in entries], dtype=np.int32)
+        counts = np.ascontiguousarray([len(t) for _, t in entries], dtype=np.int32)
+        toks = np.ascontiguousarray(np.concatenate([np.asarray(t, dtype=np.int32) for _, t in entries]))
+        if any(not 0 <= w < n for n, ws in zip(counts, want) for w in ws):
+            raise ValueError("a wanted place lies outside its entry's tokens")
+        starts = np.concatenate([[0], np.cumsum(counts)[:-1]])
+        rows = np.asarray([int(s0) + int(w) for s0, ws in zip(starts, want) for w in ws], dtype=np.int32)
+        uniq, inverse = np.unique(rows, return_inverse=True)
+        uniq = np.ascontiguousarray(uniq, dtype=np.int32)
+        n = uniq.size
+        out = np.zeros((n, self.model.cfg.vocab), dtype=np.float32) if want_logits else None
+        nxt = np.zeros(n, dtype=np.int32)
+        _lib.check(self.lib.b200_batch_step(self._h, len(entries), seqs.ctypes.data, counts.ctypes.data,
+                                            toks.ctypes.data, n, uniq.ctypes.data,
+                                            out.ctypes.data if want_logits else None, nxt.ctypes.data))
+        return (out[inverse] if want_logits else None), nxt[inverse]
 
     def last_ms(self) -> float:
         return float(self.lib.b200_batch_last_ms(self._h))

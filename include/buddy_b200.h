@@ -53,7 +53,8 @@ enum { B200_F32 = 0, B200_F16 = 1, B200_BF16 = 2 };
 enum {
   B200_W_F32 = 0, /* f32, row n = output channel, K contiguous            */
   B200_W_I8 = 1,  /* int8, per-output-channel scale                       */
-  B200_W_U4 = 2   /* 4-bit, value = nibble - 8, one scale per `group` k    */
+  B200_W_U4 = 2,  /* 4-bit, value = nibble - 8, one scale per `group` k    */
+  B200_W_BF16 = 3 /* bfloat16, row n = output channel, K contiguous        */
 };
 
 /* ------------------------------------------------------------------------
@@ -270,6 +271,47 @@ enum {
 };
 
 int b200_model_create(const b200_model_config *cfg, b200_model **out);
+
+/* ---- models given as a list of described layers ----------------------------
+ * A decoder whose layers differ: each layer names its token mixer and its
+ * feed-forward with their sizes and constants.  A layer is a parallel block,
+ * x += mixer(h) + ff(h) with h = RMSNorm(x); the output is RMSNorm and the
+ * transposed embedding table.  (No counterpart in buddy-mlir.)  The handle is
+ * an ordinary b200_model: decode, generate, prefill and the batch calls take
+ * it; tensors are loaded by name (b200_model_set_tensor). */
+enum { B200_MIX_LATENT = 0 };
+enum { B200_FF_NONE = 0, B200_FF_GATED = 1, B200_FF_EXPERTS = 2 };
+typedef struct {
+  int32_t mixer;     /* B200_MIX_LATENT: attention over a cached low-rank latent
+                      * with a rotated key part that all heads share           */
+  int32_t heads, dim, rot_dim, vdim; /* per head: unrotated and rotated query /
+                      * key sizes, value size (rotation: interleaved pairs)    */
+  int32_t kv_rank;   /* latent size                                            */
+  int32_t window;    /* sliding window in tokens, 0: everything before         */
+  int32_t kv_from;   /* attend to that earlier layer's cache, -1: own cache    */
+  float scale, rot_base;
+  int32_t ff_kind;   /* B200_FF_*                                              */
+  int32_t ff;        /* width of the feed-forward, or of one expert            */
+  int32_t experts, top;
+  float limit, gate_slope, up_offset; /* g = min(g, limit), u = clamp(u, -limit, limit),
+                      * g * sigmoid(gate_slope * g) * (u + up_offset)          */
+} b200_layer_config;
+/* cfg: hidden, n_layers, vocab, max_len and eps are read.  dtype: B200_BF16
+ * (weights, cache and matrix operands in bfloat16; norms, router, softmax,
+ * residual and all sums in f32) or B200_F32 (everything in f32). */
+int b200_model_create_layered(const b200_model_config *cfg,
+                              const b200_layer_config *layers, int dtype,
+                              b200_model **out);
+/* A named tensor from HOST memory, row-major [rows, cols] = [out, in] (vectors:
+ * rows = 1), dtype B200_BF16 or B200_F32.  Names: "embed", "final.norm", and
+ * per layer i "l<i>.norm1", "l<i>.mix.{q,dkv,dkv.norm,uk,uv,o}",
+ * "l<i>.mlp.{gate,up,down}" or "l<i>.mlp.router" and
+ * "l<i>.mlp.e<j>.{gate,up,down}". */
+int b200_model_set_tensor(b200_model *m, const char *name, int dtype,
+                          const void *host, int64_t rows, int64_t cols);
+/* Residual stream of the rows of the last prefill / batch call of such a model
+ * (after its last layer), host [n][hidden]; n must be that call's row count. */
+int b200_model_read_residual(b200_model *m, float *host, int n);
 void b200_model_destroy(b200_model *m);
 /* Upload a float vector / table from HOST memory (full, unsharded tensor). */
 int b200_model_set_vector(b200_model *m, int layer, int slot,
@@ -394,6 +436,14 @@ int b200_batch_prefill(b200_batch *b, int seq, const int32_t *tokens, int n,
 int b200_batch_decode(b200_batch *b, int n, const int *seqs,
                       const int32_t *tokens, float *logits_host,
                       int32_t *next_tokens);
+/* One step of a mixed batch: entry i brings counts[i] >= 1 next tokens of sequence
+ * seqs[i] (distinct; `tokens` holds them back to back).  Logits come back for the n_want
+ * flattened rows `want` (ascending): logits_host [n_want, vocab] or NULL, next_tokens
+ * [n_want] (first maximum) or NULL. */
+int b200_batch_step(b200_batch *b, int n_entries, const int *seqs,
+                    const int *counts, const int32_t *tokens, int n_want,
+                    const int32_t *want, float *logits_host,
+                    int32_t *next_tokens);
 float b200_batch_last_ms(const b200_batch *b);
 /* Timing of the last decode/generate call, CUDA events on the session's
  * stream (ms). */
