@@ -1800,6 +1800,7 @@ int b200_model_prefill(b200_model *m, const int32_t *tokens, int n_tokens, int p
     B200_CUDA(cudaStreamSynchronize(m->stream));
     B200_CUDA(cudaEventElapsedTime(&m->last_ms, m->ev0, m->ev1));
     m->rows_fresh = false;
+    if (int rc = layered_status(m)) return rc;
     if (next_token)
       *next_token = nxt.back();
     return B200_OK;
@@ -1867,7 +1868,7 @@ static int batch_rows(b200_batch *b, int M, const int32_t *tokens, const int32_t
     B200_CUDA(cudaEventRecord(m->ev1, st));
     B200_CUDA(cudaStreamSynchronize(st));
     B200_CUDA(cudaEventElapsedTime(&b->last_ms, m->ev0, m->ev1));
-    return B200_OK;
+    return layered_status(m);
   }
   // A w8a8 projection scales its whole activation tensor: rows of unrelated sequences in one
   // batch would share that scale, and each sequence's result would depend on its neighbours.

@@ -88,9 +88,7 @@ struct LayeredWs {             // activations of up to `rows` rows
   // tensor-core path
   bf16 *h16 = nullptr, *cat16 = nullptr, *q16 = nullptr, *x16 = nullptr, *mid16 = nullptr;
   float *expert_y = nullptr;
-  int32_t *perm = nullptr, *place = nullptr, *tiles = nullptr, *counts = nullptr;
-  bf16 *keys16 = nullptr, *kv16 = nullptr;   // a segment's cache rows, and their expanded keys and values
-  int64_t key_rows = 0;
+  int32_t *place = nullptr, *tiles = nullptr, *counts = nullptr;
 };
 struct LayeredState {
   int dtype = B200_F32;
@@ -101,6 +99,7 @@ struct LayeredState {
   std::vector<void *> owned;
   int32_t *zero = nullptr;     // sequence 0, page 0: the session's block table
   int ldp = 0, ldc = 0, ldq = 0, max_mid = 0, max_slots = 0, max_ff = 0, max_top = 0, max_experts = 0;
+  int max_q = 0, max_row = 0, max_kv = 0;
   int window = 0;              // the widest window of all layers, 0: some layer sees everything
   LayeredWs one, many;         // the captured decode step's rows, and everything else's
   float *x_want = nullptr;     // rows whose logits are asked for
@@ -108,8 +107,9 @@ struct LayeredState {
   float *logits = nullptr;
   int32_t *want = nullptr, *next = nullptr;
   int want_cap = 0;
-  void *gemm_ws = nullptr;
-  int64_t gemm_ws_bytes = 0;
+  void *gemm_ws = nullptr;     // error word, split-k partial tiles
+  bf16 *keys16 = nullptr, *kv16 = nullptr;   // a prompt segment's cache rows, and their expanded keys and values
+  int64_t key_rows = 0;
 };
 struct RowSegment {            // consecutive rows of one sequence
   int row0, n, seq, pos0;
@@ -203,6 +203,7 @@ int layered_issue_step(b200_model *m, cudaStream_t st); // one decode step of th
 int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row_seq, const int32_t *row_pos,
                  const int32_t *table_dev, int table_stride, int page, void *const *pools, int max_ctx, int n_want,
                  const int32_t *want, float *logits_host, int32_t *next_host);
+int layered_status(b200_model *m);                      // after a synchronise: did a bounded wait give up?
 int layered_clear_cache(b200_model *m);
 int64_t layered_step_bytes(const b200_model *m, int ctx);
 } // namespace b200

@@ -35,6 +35,27 @@ __global__ void embed_table_kernel(const T *table, int64_t ld, const int32_t *to
     x[(int64_t)blockIdx.x * H + i] = to_float(src[i]);
 }
 
+// h = RMSNorm(x[rows ? rows[m] : m]) as bf16 rows of ldh (zero beyond H): a CTA per row
+__global__ void __launch_bounds__(256)
+norm_rows_kernel(const float *x, const int32_t *rows, int H, const float *norm_w, float eps, bf16 *h, int64_t ldh) {
+  __shared__ float s_red[8];
+  const int m = blockIdx.x;
+  const float *src = x + (int64_t)(rows ? rows[m] : m) * H;
+  float s = 0.f;
+  for (int k = threadIdx.x; k < H; k += 256)
+    s = fmaf(src[k], src[k], s);
+  s = warp_sum(s);
+  if ((threadIdx.x & 31) == 0)
+    s_red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < 8; ++w)
+    t += s_red[w];
+  const float r = 1.0f / sqrtf(t / (float)H + eps);
+  for (int k = threadIdx.x; k < ldh; k += 256)
+    h[(int64_t)m * ldh + k] = __float2bfloat16_rn(k < H ? src[k] * r * norm_w[k] : 0.f);
+}
+
 __global__ void gather_rows_kernel(const float *x, const int32_t *rows, float *y, int H) {
   const float *src = x + (int64_t)rows[blockIdx.x] * H;
   for (int i = threadIdx.x; i < H; i += blockDim.x)
@@ -159,6 +180,9 @@ int build_layer(LayeredState *s, LayeredLayer &L, int i, int W) {
   s->ldp = std::max(s->ldp, (int)pad_to(L.plain, 4));
   s->ldc = std::max(s->ldc, (int)L.out.ld);
   s->ldq = std::max(s->ldq, d.heads * (d.rank + d.rot));
+  s->max_q = std::max(s->max_q, nq);
+  s->max_row = std::max(s->max_row, (int)d.row);
+  s->max_kv = std::max(s->max_kv, (int)pad_to(L.ukv.N, 8));
   if (experts) {
     s->max_mid = std::max(s->max_mid, c.top * c.ff);
     s->max_top = std::max(s->max_top, c.top);
@@ -167,6 +191,12 @@ int build_layer(LayeredState *s, LayeredLayer &L, int i, int W) {
   }
   return B200_OK;
 }
+
+// From this many rows on a bfloat16 model contracts on the tensor cores; a run of consecutive
+// rows of one sequence of this length expands its keys (latent_prefill.cu).
+constexpr int kDenseRows = 9, kExpandRows = 17;
+
+bool dense(const LayeredState *s, int M) { return s->dtype == B200_BF16 && M >= kDenseRows; }
 
 // Activations for up to `rows` rows, contexts up to `ctx` positions.
 int reserve(b200_model *m, LayeredWs &ws, int rows, int ctx) {
@@ -195,6 +225,21 @@ int reserve(b200_model *m, LayeredWs &ws, int rows, int ctx) {
   if (!rc) rc = own_array(o, &ws.row_seq, rows);
   if (!rc) rc = own_array(o, &ws.row_pos, rows);
   if (!rc) rc = own_array(o, &ws.tokens, rows);
+  if (dense(s, rows)) {
+    const int64_t slots = (int64_t)rows * s->max_top;
+    if (!rc) rc = own_array(o, &ws.h16, rows * pad_to(W, 8));
+    if (!rc) rc = own_array(o, &ws.cat16, (int64_t)rows * s->ldc);
+    if (!rc) rc = own_array(o, &ws.q16, (int64_t)rows * s->max_q);
+    if (s->max_top > 0) {
+      if (!rc) rc = own_array(o, &ws.x16, slots * pad_to(W, 8));
+      if (!rc) rc = own_array(o, &ws.mid16, slots * pad_to(s->max_ff, 8));
+      if (!rc) rc = own_array(o, &ws.expert_y, slots * W);
+      if (!rc) rc = own_array(o, &ws.place, slots);
+      if (!rc) rc = own_array(o, &ws.counts, s->max_experts + 4);
+      if (!rc) rc = own_array(o, &ws.tiles, 4 * (int64_t)experts_max_tiles((int)slots, s->max_experts));
+    }
+    if (!rc && !s->gemm_ws) rc = own_alloc(s->owned, &s->gemm_ws, (size_t)gemm_bf16_workspace_bytes());
+  }
   if (rc) {
     release(ws.owned);
     ws = LayeredWs();
@@ -202,6 +247,13 @@ int reserve(b200_model *m, LayeredWs &ws, int rows, int ctx) {
   }
   ws.rows = rows;
   ws.ctx = ctx;
+  return B200_OK;
+}
+
+int norm_rows_launch(const float *x, const int32_t *rows, int H, int M, const float *norm_w, float eps, bf16 *h, int64_t ldh,
+                     cudaStream_t st) {
+  norm_rows_kernel<<<M, 256, 0, st>>>(x, rows, H, norm_w, eps, h, ldh);
+  B200_LAUNCH_CHECK();
   return B200_OK;
 }
 
@@ -236,6 +288,116 @@ int row_layers(b200_model *m, LayeredWs &ws, float *x, int M, const CacheView &c
   return B200_OK;
 }
 
+// Room for a segment's gathered cache rows and expanded keys.
+int reserve_keys(b200_model *m, int64_t n) {
+  LayeredState *s = m->lay;
+  if (n <= s->key_rows)
+    return B200_OK;
+  B200_CUDA(cudaStreamSynchronize(m->stream));
+  cudaFree(s->keys16);
+  cudaFree(s->kv16);
+  s->keys16 = s->kv16 = nullptr;
+  s->key_rows = 0;
+  if (int rc = dev_alloc((void **)&s->keys16, (size_t)n * s->max_row * 2)) return rc;
+  if (int rc = dev_alloc((void **)&s->kv16, (size_t)n * s->max_kv * 2)) return rc;
+  s->key_rows = n;
+  return B200_OK;
+}
+
+// The attention of one layer for all rows, bf16: long runs of a sequence over expanded keys,
+// what lies between them in the single-query form.
+int dense_attention(b200_model *m, LayeredWs &ws, LayeredLayer &L, int M, const CacheView &cv,
+                    const std::vector<RowSegment> &segs, void *pool, int max_ctx, cudaStream_t st) {
+  LayeredState *s = m->lay;
+  const LatentDims &d = L.d;
+  auto singles = [&](int r0, int n) {
+    CacheView c = cv;
+    c.row_seq += r0;
+    c.row_pos += r0;
+    const int splits = latent_splits(d, n, max_ctx);
+    if (int rc = latent_prep_launch(s->dtype, d, ws.proj + (int64_t)r0 * s->ldp, s->ldp, n, L.uk, L.inv_freq, ws.qabs,
+                                    false, 0, nullptr, 0.f, pool, c, st))
+      return rc;
+    if (int rc = latent_attend_launch(s->dtype, d, ws.qabs, n, pool, c, splits, max_ctx, ws.part, st)) return rc;
+    return latent_value_launch(s->dtype, d, ws.part, n, splits, L.uv, ws.cat16 + (int64_t)r0 * s->ldc, s->ldc, true, st);
+  };
+  int begin = 0;                         // first row not yet attended for
+  for (const RowSegment &g : segs) {
+    if (g.n < kExpandRows || !latent_prefill_takes(d))
+      continue;
+    if (g.row0 > begin)
+      if (int rc = singles(begin, g.row0 - begin)) return rc;
+    begin = g.row0 + g.n;
+    const int first = d.window > 0 ? std::max(0, g.pos0 - d.window + 1) : 0;
+    const int keys = g.pos0 + g.n - first;
+    if (int rc = reserve_keys(m, keys)) return rc;
+    if (int rc = latent_gather_launch(d, pool, cv, g.seq, first, keys, s->keys16, st)) return rc;
+    GemmBf16 e;
+    e.A = s->keys16; e.lda = d.row; e.M = keys; e.w = L.ukv; e.C16 = s->kv16; e.ldc = pad_to(L.ukv.N, 8);
+    if (int rc = gemm_bf16_launch(e, s->gemm_ws, st)) return rc;
+    if (int rc = latent_query_launch(d, ws.proj + (int64_t)g.row0 * s->ldp, s->ldp, g.n, L.inv_freq, cv.row_pos + g.row0,
+                                     ws.q16, st))
+      return rc;
+    if (int rc = latent_prefill_launch(d, ws.q16, g.n, g.pos0, s->keys16, s->kv16, e.ldc, first,
+                                       ws.cat16 + (int64_t)g.row0 * s->ldc, s->ldc, st))
+      return rc;
+  }
+  return begin < M ? singles(begin, M - begin) : B200_OK;
+}
+
+// All layers over M rows on the tensor cores (bfloat16 models, more than a handful of rows).
+int dense_layers(b200_model *m, LayeredWs &ws, float *x, int M, const CacheView &cv, const std::vector<RowSegment> &segs,
+                 void *const *pools, int max_ctx, cudaStream_t st) {
+  LayeredState *s = m->lay;
+  const int W = m->cfg.hidden;
+  const int64_t ldh = pad_to(W, 8);
+  for (LayeredLayer &L : s->layers) {
+    const b200_layer_config &c = L.cfg;
+    void *pool = pools[L.source];
+    if (int rc = norm_rows_launch(x, nullptr, W, M, L.norm, m->cfg.eps, ws.h16, ldh, st)) return rc;
+    GemmBf16 in;
+    in.A = ws.h16; in.lda = ldh; in.M = M; in.w = L.in; in.w.N = L.plain; in.C = ws.proj; in.ldc = s->ldp;
+    if (int rc = gemm_bf16_launch(in, s->gemm_ws, st)) return rc;
+    if (L.own())
+      if (int rc = latent_store_launch(L.d, ws.proj, s->ldp, M, L.off_down, L.down_norm, m->cfg.eps, L.inv_freq, pool, cv, st))
+        return rc;
+    if (int rc = dense_attention(m, ws, L, M, cv, segs, pool, max_ctx, st)) return rc;
+    if (c.ff_kind == B200_FF_GATED) {
+      GemmBf16 g;
+      g.A = ws.h16; g.lda = ldh; g.M = M; g.w = L.in;
+      g.w.w = (bf16 *)L.in.w + (int64_t)L.plain * L.in.ld;
+      g.w.N = 2 * c.ff;
+      g.C16 = ws.cat16 + L.att; g.ldc = s->ldc; g.pairs = true; g.gate = L.gate;
+      if (int rc = gemm_bf16_launch(g, s->gemm_ws, st)) return rc;
+    }
+    GemmBf16 o;
+    o.A = ws.cat16; o.lda = s->ldc; o.M = M; o.w = L.out; o.C = x; o.ldc = W; o.add = true;
+    if (c.ff_kind == B200_FF_EXPERTS) {
+      const int slots = M * c.top;
+      int4 *tiles = (int4 *)ws.tiles;
+      int32_t *n_tiles = ws.counts + s->max_experts;
+      const int64_t ldm = pad_to(c.ff, 8);
+      if (int rc = experts_sort_launch(ws.proj + L.off_router, s->ldp, c.experts, c.top, M, ws.h16, ldh, ws.ids, ws.weight,
+                                       ws.counts, tiles, n_tiles, ws.place, ws.x16, st))
+        return rc;
+      GemmBf16 g;
+      g.A = ws.x16; g.lda = ldh; g.M = slots; g.w = L.expert_in; g.C16 = ws.mid16; g.ldc = ldm; g.pairs = true;
+      g.gate = L.gate; g.tiles = tiles; g.n_tiles = n_tiles; g.groups = c.experts;
+      g.max_tiles = experts_max_tiles(slots, c.experts);
+      if (int rc = gemm_bf16_launch(g, s->gemm_ws, st)) return rc;
+      GemmBf16 dn;
+      dn.A = ws.mid16; dn.lda = ldm; dn.M = slots; dn.w = L.expert_out; dn.C = ws.expert_y; dn.ldc = W;
+      dn.tiles = tiles; dn.n_tiles = n_tiles; dn.groups = c.experts; dn.max_tiles = g.max_tiles;
+      if (int rc = gemm_bf16_launch(dn, s->gemm_ws, st)) return rc;
+      if (int rc = gemm_bf16_launch(o, s->gemm_ws, st)) return rc;
+      if (int rc = experts_combine_launch(x, W, c.top, M, ws.expert_y, ws.place, ws.weight, st)) return rc;
+    } else if (int rc = gemm_bf16_launch(o, s->gemm_ws, st)) {
+      return rc;
+    }
+  }
+  return B200_OK;
+}
+
 int embed_tokens(b200_model *m, const int32_t *tokens, float *x, int M, cudaStream_t st) {
   LayeredState *s = m->lay;
   const int W = m->cfg.hidden;
@@ -249,6 +411,13 @@ int embed_tokens(b200_model *m, const int32_t *tokens, float *x, int M, cudaStre
 
 int head(b200_model *m, const float *x, int n, float *logits, cudaStream_t st) {
   LayeredState *s = m->lay;
+  if (dense(s, n) && s->gemm_ws) {
+    const int64_t ldh = pad_to(m->cfg.hidden, 8);
+    if (int rc = norm_rows_launch(x, nullptr, m->cfg.hidden, n, s->final_norm, m->cfg.eps, s->h_want, ldh, st)) return rc;
+    GemmBf16 g;
+    g.A = s->h_want; g.lda = ldh; g.M = n; g.w = s->embed; g.C = logits; g.ldc = m->cfg.vocab;
+    return gemm_bf16_launch(g, s->gemm_ws, st);
+  }
   return gemv_rows_launch(s->dtype, s->embed, x, m->cfg.hidden, n, s->final_norm, m->cfg.eps, logits, m->cfg.vocab, false,
                           m->cfg.vocab, nullptr, 0, Gate{}, st);
 }
@@ -269,7 +438,7 @@ void layered_destroy(b200_model *m) {
   release(s->many.owned);
   release(s->owned);
   cudaFree(s->x_want); cudaFree(s->h_want); cudaFree(s->logits); cudaFree(s->want); cudaFree(s->next);
-  cudaFree(s->gemm_ws);
+  cudaFree(s->keys16); cudaFree(s->kv16);
   delete s;
   m->lay = nullptr;
 }
@@ -327,7 +496,19 @@ int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row
     B200_CUDA(cudaMemcpyAsync(ws.row_pos, row_pos + m0, (size_t)n * 4, cudaMemcpyHostToDevice, st));
     const CacheView cv{ws.row_seq, ws.row_pos, table_dev, table_stride, page};
     if (int rc = embed_tokens(m, ws.tokens, ws.x, n, st)) return rc;
-    if (int rc = row_layers(m, ws, ws.x, n, cv, pools, max_ctx, st)) return rc;
+    if (dense(s, n)) {
+      std::vector<RowSegment> segs;
+      for (int r = 0; r < n; ++r) {
+        const int32_t seq = row_seq[m0 + r], pos = row_pos[m0 + r];
+        if (!segs.empty() && segs.back().seq == seq && segs.back().pos0 + segs.back().n == pos)
+          segs.back().n += 1;
+        else
+          segs.push_back(RowSegment{r, 1, seq, pos});
+      }
+      if (int rc = dense_layers(m, ws, ws.x, n, cv, segs, pools, max_ctx, st)) return rc;
+    } else if (int rc = row_layers(m, ws, ws.x, n, cv, pools, max_ctx, st)) {
+      return rc;
+    }
     local.clear();
     for (int k = done; k < n_want && want[k] < m0 + n; ++k)
       local.push_back(want[k] - m0);
@@ -348,6 +529,19 @@ int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row
       B200_CUDA(cudaMemcpyAsync(next_host, s->next, (size_t)n_want * 4, cudaMemcpyDeviceToHost, st));
   }
   return B200_OK;
+}
+
+int layered_status(b200_model *m) {
+  LayeredState *s = m->lay;
+  if (!s->gemm_ws)
+    return B200_OK;
+  int code = 0;
+  B200_CUDA(cudaMemcpyAsync(&code, s->gemm_ws, 4, cudaMemcpyDeviceToHost, m->stream));
+  B200_CUDA(cudaStreamSynchronize(m->stream));
+  if (code == 0)
+    return B200_OK;
+  B200_CUDA(cudaMemsetAsync(s->gemm_ws, 0, 4, m->stream));
+  return fail(B200_ECUDA, "gemm_bf16: a bounded wait gave up (code %d)", code);
 }
 
 int64_t layered_step_bytes(const b200_model *m, int ctx) {

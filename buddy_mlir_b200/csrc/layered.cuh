@@ -96,8 +96,42 @@ int latent_value_launch(int dtype, const LatentDims &d, const float *scratch, in
                         void *out, int64_t ldo, bool out_bf16, cudaStream_t st);
 int latent_limits(const LatentDims &d);   // 0, or an error for sizes the kernels do not take
 
-// rows_ops in layered.cu
-int place_rows_launch(int src_dtype, const void *src, int rows, int cols, int dst_dtype, void *dst, int64_t ld, int64_t row0,
-                      int64_t row_step, int64_t col0, cudaStream_t st);
+// latent_prefill.cu: many consecutive queries of one sequence, bf16
+int latent_store_launch(const LatentDims &d, const float *proj, int64_t ldp, int M, int off_down, const float *norm_w,
+                        float eps, const float *inv_freq, void *pool, const CacheView &cv, cudaStream_t st);
+int latent_query_launch(const LatentDims &d, const float *proj, int64_t ldp, int M, const float *inv_freq,
+                        const int32_t *row_pos, bf16 *q, cudaStream_t st);
+int latent_gather_launch(const LatentDims &d, const void *pool, const CacheView &cv, int seq, int first, int n, bf16 *rows,
+                         cudaStream_t st);
+bool latent_prefill_takes(const LatentDims &d);
+int latent_prefill_launch(const LatentDims &d, const bf16 *q, int n, int pos0, const bf16 *rows, const bf16 *kv, int64_t ldkv,
+                          int first, bf16 *out, int64_t ldo, cudaStream_t st);
+
+// gemm_bf16.cu
+struct GemmBf16 {
+  const bf16 *A = nullptr;     // [M][lda], K used elements per row
+  int64_t lda = 0;
+  int M = 0;
+  RowMatrix w;                 // bf16 rows
+  float *C = nullptr;          // result as f32 or as bf16, rows of ldc
+  bf16 *C16 = nullptr;
+  int64_t ldc = 0;
+  bool add = false;            // C += (f32 only)
+  bool pairs = false;          // rows (2j, 2j + 1) of w are (gate_j, up_j): N / 2 gated columns
+  Gate gate{};
+  const int4 *tiles = nullptr; // grouped: row tiles (group, first row, rows), at most max_tiles of them
+  const int32_t *n_tiles = nullptr;
+  int max_tiles = 0, groups = 1;   // w holds `groups` matrices of N / groups rows
+};
+int64_t gemm_bf16_workspace_bytes();
+int gemm_bf16_launch(const GemmBf16 &g, void *workspace, cudaStream_t st);
+
+// experts.cu
+int experts_max_tiles(int slots, int experts);
+int experts_sort_launch(const float *z, int64_t ldz, int experts, int top, int M, const bf16 *h, int64_t ldh, int32_t *ids,
+                        float *weight, int32_t *counts, int4 *tiles, int32_t *n_tiles, int32_t *place, bf16 *sorted,
+                        cudaStream_t st);
+int experts_combine_launch(float *x, int W, int top, int M, const float *y, const int32_t *place, const float *weight,
+                           cudaStream_t st);
 
 } // namespace b200
