@@ -517,6 +517,128 @@ def run_batch_only(args):
     print(json.dumps(batch_numbers(blob, args.steps, args.warmup)))
 
 
+# Models of described layers beside the uniform attention model of the same width, depth, head count
+# and (active) feed-forward width.  name: (hidden, heads, kv heads of the other, dense ff, experts, top, expert ff)
+LAYERED_SHAPES = {
+    "1p5b_dense": (1536, 12, 2, 8960, 0, 0, 0),
+    "2k_experts": (2048, 16, 4, 8448, 64, 6, 1408),
+    "8b_dense": (4096, 32, 8, 12288, 0, 0, 0),
+}
+LAYERED = {"layers": 4, "vocab": 32768, "window": 1024, "rank": 512, "rot": 64, "dim": 128, "vdim": 128,
+           "prefill": 2048, "context": 1024, "batch": 64}
+
+
+def layered_model(name, window=None):
+    """A Talazen of LAYERED_SHAPES with seeded weights (repeated tiles of one seeded pool: values do
+    not matter for the time), every second layer attending to the cache of the one before it."""
+    from buddy_mlir_b200 import talazen
+    from buddy_mlir_b200.session import ModelSession
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    H, heads, _, ff, experts, top, eff = LAYERED_SHAPES[name]
+    L = LAYERED
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+    layers = []
+    for i in range(L["layers"]):
+        m = {"heads": heads, "dim": L["dim"], "rot_dim": L["rot"], "vdim": L["vdim"], "kv_rank": L["rank"],
+             "rot": {"base": 10000.0, "dims": L["rot"]}, "mask": {"size": window or L["window"]},
+             "scale": (L["dim"] + L["rot"]) ** -0.5}
+        if i % 2:
+            m["kv_from"] = i - 1
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": moe if experts else dense})
+    cfg = {"architecture": "Talazen", "width": H, "vocab": L["vocab"], "norm": {"eps": 1e-5}, "layers": layers}
+    import plain_talazen
+    pool = np.random.default_rng(SEED_W).standard_normal(1 << 22).astype(np.float32) * 0.02
+    pool16 = (pool.view(np.uint32) >> 16).astype(np.uint16)
+    big = np.tile(pool16, 64)
+    s = ModelSession(talazen.parse(cfg, "bfloat16", 4096))
+    s.load_named({k: (np.ones(shape, np.float32) if len(shape) == 1 else big[:shape[0] * shape[1]].reshape(shape))
+                  for k, shape in plain_talazen.tensor_shapes(cfg).items()})
+    return s
+
+
+def uniform_model(name):
+    """The int8 uniform-attention model of the same width, depth, heads and active feed-forward."""
+    from buddy_mlir_b200 import _lib
+    from buddy_mlir_b200.config import ModelConfig
+    from buddy_mlir_b200.session import ModelSession
+    from buddy_mlir_b200.synthetic import tensor_list
+    H, heads, kvh, ff, _, _, _ = LAYERED_SHAPES[name]
+    cfg = ModelConfig(name, H, LAYERED["layers"], heads, kvh, 128, ff, LAYERED["vocab"], 4096)
+    pool = np.random.default_rng(SEED_W).standard_normal(1 << 22).astype(np.float32) * 0.02
+    big = np.tile(pool, 64)
+    s = ModelSession(cfg)
+    s.load_tensors({(n, l): (np.ones(shape, np.float32) if "norm" in n else big[:int(np.prod(shape))].reshape(shape))
+                    for n, l, shape in tensor_list(cfg)}, quantize_to="w8")
+    return s
+
+
+def session_numbers(s, steps=64):
+    """Prefill, single-sequence decode and batched decode of a session (CUDA events)."""
+    import torch
+    from buddy_mlir_b200.session import BatchSession
+    L, cfg = LAYERED, s.cfg
+    rng = np.random.default_rng(SEED_P)
+    n, ctx, B = L["prefill"], L["context"], L["batch"]
+    s.prefill_rows(rng.integers(0, cfg.vocab, ctx), 0, all_rows=False)
+    s.generate(3, 8)
+    s.generate(5, steps)
+    decode = s.last_ms() / steps
+    per_page = 64
+    bs = BatchSession(s, B + 1, per_page, (B + 2) * ((ctx + steps) // per_page + 2) + n // per_page, max(n, ctx + steps) + 64)
+    ms = []
+    for i in range(4):
+        q = bs.add()
+        if i == 3:
+            torch.cuda.profiler.start()
+        bs.prefill(q, rng.integers(0, cfg.vocab, n), want_logits=False)
+        torch.cuda.profiler.stop()
+        ms.append(bs.last_ms())
+        bs.remove(q)
+    prefill = min(ms[1:])
+    seqs = [bs.add() for _ in range(B)]
+    for q in seqs:
+        bs.prefill(q, rng.integers(0, cfg.vocab, ctx), want_logits=False)
+    toks, ms = [7] * B, []
+    for i in range(3 + 16):
+        if i == 18:
+            torch.cuda.profiler.start()
+        _, toks = bs.decode(seqs, toks, want_logits=False)
+        torch.cuda.profiler.stop()
+        ms.append(bs.last_ms())
+    batched = float(np.mean(ms[3:]))
+    bs.close()
+    hbm, _ = peaks()
+    step_bytes = s.step_bytes(ctx + steps // 2)
+    return {"prefill": {"rows": n, "ms": prefill, "tokens_per_s": n / prefill * 1e3},
+            "decode": {"context": ctx, "ms": decode, "tokens_per_s": 1e3 / decode, "bytes_per_step": step_bytes,
+                       "hbm_frac": step_bytes / decode / 1e6 / hbm},
+            "batched_decode": {"sequences": B, "context": ctx, "ms": batched, "tokens_per_s": B / batched * 1e3}}
+
+
+def run_layered_only(args):
+    """--layered: prefill and decode of models of described layers (Talazen, bfloat16) at the sizes of
+    LAYERED_SHAPES, beside the uniform int8 model of equal size (one JSON line)."""
+    import torch
+    from buddy_mlir_b200 import _lib
+    _lib.load()
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device; the library has no CPU path")
+    torch.cuda.set_device(0)
+    out = {}
+    for name in ([args.layered_shape] if args.layered_shape else LAYERED_SHAPES):
+        out[name] = {}
+        for kind, make in (("talazen_bf16", layered_model), ("uniform_int8", uniform_model)):
+            if args.layered_kind and args.layered_kind != kind:
+                continue
+            s = make(name)
+            out[name][kind] = session_numbers(s)
+            s.close()
+    print(json.dumps({"layered": out, "sizes": LAYERED,
+                      "shapes": {k: dict(zip(("hidden", "heads", "kv_heads_uniform", "ff_dense_or_active", "experts", "top", "expert_ff"), v))
+                                 for k, v in LAYERED_SHAPES.items()}, "data": "synthetic, seeded weights"}))
+
+
 def run_gemv_only(args):
     """--gemv-only: just the isolated GEMV sweep (one JSON line); --gemv-shape picks one shape,
     which keeps a profiler capture of that kernel small."""
@@ -649,6 +771,10 @@ def main():
     ap.add_argument("--gemm-only", action="store_true", help="run only the isolated dense-GEMM sweep (tcgen05 path)")
     ap.add_argument("--batch-only", action="store_true", help="batched decode (64 sequences, paged KV) + a 2048-token prefill")
     ap.add_argument("--w8a8-only", action="store_true", help="the w8a8 arithmetic on the 1.5B int8 model: prefill and decode")
+    ap.add_argument("--layered", action="store_true",
+                    help="models of described layers (Talazen) beside the uniform model of equal size: prefill, decode, batched decode")
+    ap.add_argument("--layered-shape", default=None, help="with --layered: one of LAYERED_SHAPES")
+    ap.add_argument("--layered-kind", default=None, help="with --layered: talazen_bf16 or uniform_int8 alone")
     ap.add_argument("--gemm-shape", default=None, help="with --gemm-only: one shape of GEMM_SHAPES")
     ap.add_argument("--resident-only", action="store_true",
                     help="skip the isolated-GEMV, end-to-end and CPU legs (for profiler captures)")
@@ -668,6 +794,8 @@ def main():
         return run_batch_only(args)
     if args.w8a8_only:
         return run_w8a8_only(args)
+    if args.layered:
+        return run_layered_only(args)
     if args.gpus == 1 and int(os.environ.get("WORLD_SIZE", "1")) == 1:
         return run_single(args)
     import bench_tp
