@@ -584,6 +584,9 @@ def session_numbers(s, steps=64):
     s.generate(3, 8)
     s.generate(5, steps)
     decode = s.last_ms() / steps
+    torch.cuda.profiler.start()      # profiler ranges: one decode step, one prefill, one batched step
+    s.generate(5, 1)
+    torch.cuda.profiler.stop()
     per_page = 64
     bs = BatchSession(s, B + 1, per_page, (B + 2) * ((ctx + steps) // per_page + 2) + n // per_page, max(n, ctx + steps) + 64)
     ms = []

@@ -9,18 +9,34 @@ namespace {
 
 constexpr int BM = 128;        // rows per tile of the grouped GEMM
 
-// one warp per row; counts[e] is the number of slots of expert e
+// a warp routes kRouteRows rows; counts[e] is the number of slots of expert e
+constexpr int kRouteRows = 2;
 __global__ void __launch_bounds__(256)
 route_rows_kernel(const float *z, int64_t ldz, int experts, int top, int M, int32_t *ids, float *weight, int32_t *counts) {
-  extern __shared__ float s_z[];
+  extern __shared__ float s_z[];   // per warp: experts logits, top weights, top ids; then the CTA's counts
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int m = blockIdx.x * 8 + warp;
-  if (m >= M)
-    return;
-  int32_t *id = ids + (int64_t)m * top;
-  route_row(z + (int64_t)m * ldz, experts, top, s_z + warp * experts, id, weight + (int64_t)m * top, lane);
-  for (int j = lane; j < top; j += 32)
-    atomicAdd(counts + id[j], 1);
+  float *sz = s_z + warp * (experts + 2 * top), *sw = sz + experts;
+  int *sid = reinterpret_cast<int *>(sw + top);
+  int *s_count = reinterpret_cast<int *>(s_z + 8 * (experts + 2 * top));
+  for (int e = threadIdx.x; e < experts; e += 256)
+    s_count[e] = 0;
+  __syncthreads();
+  for (int r = 0; r < kRouteRows; ++r) {
+    const int m = (blockIdx.x * 8 + warp) * kRouteRows + r;
+    if (m >= M)
+      break;
+    route_row(z + (int64_t)m * ldz, experts, top, sz, sid, sw, lane);
+    for (int j = lane; j < top; j += 32) {
+      ids[(int64_t)m * top + j] = sid[j];
+      weight[(int64_t)m * top + j] = sw[j];
+      atomicAdd(s_count + sid[j], 1);
+    }
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < experts; e += 256)
+    if (s_count[e] > 0)
+      atomicAdd(counts + e, s_count[e]);
 }
 
 // counts -> first sorted row of every expert (left in counts as a cursor) and the tile table
@@ -70,12 +86,36 @@ sort_rows_kernel(const bf16 *h, int64_t ldh, int top, int slots, const int32_t *
 // x[m] += sum over j of weight[m, j] * y[place[m, j]]
 __global__ void __launch_bounds__(256)
 combine_experts_kernel(float *x, int W, int top, const float *y, const int32_t *place, const float *weight) {
-  const int m = blockIdx.x;
-  for (int n = threadIdx.x; n < W; n += 256) {
-    float s = 0.f;
-    for (int j = 0; j < top; ++j)
-      s = fmaf(weight[(int64_t)m * top + j], y[(int64_t)place[(int64_t)m * top + j] * W + n], s);
-    x[(int64_t)m * W + n] += s;
+  extern __shared__ float s_w[];   // top weights, top places
+  int *s_p = reinterpret_cast<int *>(s_w + top);
+  const int64_t m = blockIdx.x;
+  for (int j = threadIdx.x; j < top; j += 256) {
+    s_w[j] = weight[m * top + j];
+    s_p[j] = place[m * top + j];
+  }
+  __syncthreads();
+  if ((W & 3) == 0) {
+    for (int n = threadIdx.x * 4; n < W; n += 1024) {
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int j = 0; j < top; ++j) {
+        const float4 v = __ldg(reinterpret_cast<const float4 *>(y + (int64_t)s_p[j] * W + n));
+        s.x = fmaf(s_w[j], v.x, s.x);
+        s.y = fmaf(s_w[j], v.y, s.y);
+        s.z = fmaf(s_w[j], v.z, s.z);
+        s.w = fmaf(s_w[j], v.w, s.w);
+      }
+      float4 *dst = reinterpret_cast<float4 *>(x + m * W + n);
+      const float4 v = *dst;
+      *dst = make_float4(v.x + s.x, v.y + s.y, v.z + s.z, v.w + s.w);
+    }
+  } else {
+    for (int n = threadIdx.x; n < W; n += 256) {
+      float s = 0.f;
+      for (int j = 0; j < top; ++j)
+        s = fmaf(s_w[j], y[(int64_t)s_p[j] * W + n], s);
+      x[m * W + n] += s;
+    }
   }
 }
 
@@ -86,8 +126,11 @@ int experts_max_tiles(int slots, int experts) { return slots / BM + (experts < s
 int experts_sort_launch(const float *z, int64_t ldz, int experts, int top, int M, const bf16 *h, int64_t ldh, int32_t *ids,
                         float *weight, int32_t *counts, int4 *tiles, int32_t *n_tiles, int32_t *place, bf16 *sorted,
                         cudaStream_t st) {
+  const size_t route_bytes = ((size_t)8 * (experts + 2 * top) + experts) * 4;
+  if (route_bytes > 40 * 1024)
+    B200_CUDA(cudaFuncSetAttribute(route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024));
   B200_CUDA(cudaMemsetAsync(counts, 0, (size_t)experts * 4, st));
-  route_rows_kernel<<<(M + 7) / 8, 256, (size_t)experts * 8 * 4, st>>>(z, ldz, experts, top, M, ids, weight, counts);
+  route_rows_kernel<<<(M + 8 * kRouteRows - 1) / (8 * kRouteRows), 256, route_bytes, st>>>(z, ldz, experts, top, M, ids, weight, counts);
   B200_LAUNCH_CHECK();
   plan_tiles_kernel<<<1, 1024, 0, st>>>(counts, experts, tiles, n_tiles);
   B200_LAUNCH_CHECK();
@@ -98,7 +141,7 @@ int experts_sort_launch(const float *z, int64_t ldz, int experts, int top, int M
 
 int experts_combine_launch(float *x, int W, int top, int M, const float *y, const int32_t *place, const float *weight,
                            cudaStream_t st) {
-  combine_experts_kernel<<<M, 256, 0, st>>>(x, W, top, y, place, weight);
+  combine_experts_kernel<<<M, 256, (size_t)top * 8, st>>>(x, W, top, y, place, weight);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

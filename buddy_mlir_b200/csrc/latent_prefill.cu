@@ -24,23 +24,35 @@ __device__ __forceinline__ void rotate(float u, float v, float angle, float &a, 
   b = v * c + u * s;
 }
 
-// a warp per row
-__global__ void __launch_bounds__(256)
-latent_store_kernel(const float *proj, int64_t ldp, int M, int off, LatentDims d, const float *norm_w, float eps,
+// a CTA of 128 threads per row
+__global__ void __launch_bounds__(128)
+latent_store_kernel(const float *proj, int64_t ldp, int off, LatentDims d, const float *norm_w, float eps,
                     const float *inv_freq, bf16 *pool, CacheView cv) {
-  const int lane = threadIdx.x & 31, m = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (m >= M)
-    return;
+  __shared__ float s_red[4];
+  const int m = blockIdx.x;
   const float *down = proj + (int64_t)m * ldp + off;
   const int pos = cv.row_pos[m];
   bf16 *row = pool + cache_row(cv, cv.row_seq[m], pos) * d.row;
+  float v[8];                    // rank <= 1024
   float s = 0.f;
-  for (int k = lane; k < d.rank; k += 32)
-    s = fmaf(down[k], down[k], s);
-  const float r = 1.0f / sqrtf(warp_sum(s) / (float)d.rank + eps);
-  for (int k = lane; k < d.rank; k += 32)
-    row[k] = __float2bfloat16_rn(down[k] * r * norm_w[k]);
-  for (int i = lane; i < d.rot / 2; i += 32) {
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int k = i * 128 + threadIdx.x;
+    v[i] = k < d.rank ? down[k] : 0.f;
+    s = fmaf(v[i], v[i], s);
+  }
+  s = warp_sum(s);
+  if ((threadIdx.x & 31) == 0)
+    s_red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  const float r = 1.0f / sqrtf((s_red[0] + s_red[1] + s_red[2] + s_red[3]) / (float)d.rank + eps);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int k = i * 128 + threadIdx.x;
+    if (k < d.rank)
+      row[k] = __float2bfloat16_rn(v[i] * r * norm_w[k]);
+  }
+  for (int i = threadIdx.x; i < d.rot / 2; i += 128) {
     float a, b;
     rotate(down[d.rank + 2 * i], down[d.rank + 2 * i + 1], (float)pos * inv_freq[i], a, b);
     row[d.rank + 2 * i] = __float2bfloat16_rn(a);
@@ -59,6 +71,17 @@ latent_query_kernel(const float *proj, int64_t ldp, LatentDims d, const float *i
   __syncthreads();
   const float *src = proj + (int64_t)m * ldp;
   bf16 *dst = q + (int64_t)m * d.heads * dq;
+  if ((d.dim & 1) == 0 && (ldp & 1) == 0) {   // pairs never straddle the two parts
+    const int hp = dq / 2;
+    for (int k = threadIdx.x; k < d.heads * hp; k += 256) {
+      const int i = k % hp - d.dim / 2;
+      float2 v = *reinterpret_cast<const float2 *>(src + 2 * k);
+      if (i >= 0)
+        v = make_float2(v.x * s_cs[i] - v.y * s_cs[half + i], v.y * s_cs[i] + v.x * s_cs[half + i]);
+      *reinterpret_cast<__nv_bfloat162 *>(dst + 2 * k) = __floats2bfloat162_rn(v.x, v.y);
+    }
+    return;
+  }
   for (int k = threadIdx.x; k < d.heads * dq; k += 256) {
     const int c = k % dq - d.dim;
     float v = src[k];
@@ -95,37 +118,12 @@ struct FlashP {
   int vec;                     // 16-byte copies possible
 };
 
-constexpr int QT = 128, KT = 64;
+constexpr int QT = 128, KT = 64, kWarps = QT / 16, kThreads = kWarps * 32;
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void *p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(src), "r"(live ? 16 : 0) : "memory");
-}
-// two f32 as packed bf16 (first in the low half), and what the rounding left
-__device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t &lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
-  hi = *reinterpret_cast<const uint32_t *>(&h);
-  lo = *reinterpret_cast<const uint32_t *>(&l);
-}
-
-// grid (query tiles, heads, value columns / DV), 8 warps of 16 queries.  DK >= dim + rot and DV:
+// grid (query tiles, heads, value columns / DV), a warp per 16 queries.  DK >= dim + rot and DV:
 // padded widths; value rows wider than DV are taken DV columns per CTA.
 template <int DK, int DV>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kThreads)
 latent_prefill_kernel(const FlashP p) {
   constexpr int LK = DK + 8, LV = DV + 8;
   extern __shared__ __align__(16) bf16 sm[];
@@ -143,7 +141,7 @@ latent_prefill_kernel(const FlashP p) {
   const int lo = d.window > 0 ? max(0, i_min - d.window + 1) : 0;
   const int tiles = (i_max - lo) / KT + 1;
 
-  for (int i = threadIdx.x; i < (QT * LK + 2 * KT * LK + 2 * KT * LV) / 8; i += 256)
+  for (int i = threadIdx.x; i < (QT * LK + 2 * KT * LK + 2 * KT * LV) / 8; i += kThreads)
     reinterpret_cast<uint4 *>(sm)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
   {
@@ -151,12 +149,12 @@ latent_prefill_kernel(const FlashP p) {
     const int rows = q_last - q0 + 1;
     if (p.vec) {
       const int cpr = dq / 8;
-      for (int i = threadIdx.x; i < rows * cpr; i += 256) {
+      for (int i = threadIdx.x; i < rows * cpr; i += kThreads) {
         const int r = i / cpr, c = (i - r * cpr) * 8;
         *reinterpret_cast<uint4 *>(s_q + r * LK + c) = *reinterpret_cast<const uint4 *>(src + (int64_t)r * d.heads * dq + c);
       }
     } else {
-      for (int i = threadIdx.x; i < rows * dq; i += 256) {
+      for (int i = threadIdx.x; i < rows * dq; i += kThreads) {
         const int r = i / dq, c = i - r * dq;
         s_q[r * LK + c] = src[(int64_t)r * d.heads * dq + c];
       }
@@ -167,7 +165,7 @@ latent_prefill_kernel(const FlashP p) {
     bf16 *kd = s_k + buf * KT * LK, *vd = s_v + buf * KT * LV;
     if (p.vec) {
       const int ck = d.dim / 8, cr = d.rot / 8, cv = vdim / 8, cpr = ck + cr + cv;
-      for (int i = threadIdx.x; i < KT * cpr; i += 256) {
+      for (int i = threadIdx.x; i < KT * cpr; i += kThreads) {
         const int r = i / cpr, c = i - r * cpr;
         const bool live = j0 + r <= i_max;
         const int64_t key = (live ? j0 + r : i_max) - p.first;
@@ -180,7 +178,7 @@ latent_prefill_kernel(const FlashP p) {
       }
     } else {
       const int cpr = dq + vdim;
-      for (int i = threadIdx.x; i < KT * cpr; i += 256) {
+      for (int i = threadIdx.x; i < KT * cpr; i += kThreads) {
         const int r = i / cpr, c = i - r * cpr;
         const bool live = j0 + r <= i_max;
         const int64_t key = (live ? j0 + r : i_max) - p.first;
@@ -322,7 +320,7 @@ template <int DK, int DV> int flash_run(const FlashP &p, cudaStream_t st) {
     if (dev >= 0 && dev < 64)
       configured[dev] = 1;
   }
-  kern<<<dim3((p.n + QT - 1) / QT, p.d.heads, (p.d.vdim + DV - 1) / DV), 256, smem, st>>>(p);
+  kern<<<dim3((p.n + QT - 1) / QT, p.d.heads, (p.d.vdim + DV - 1) / DV), kThreads, smem, st>>>(p);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -337,7 +335,7 @@ bool latent_prefill_takes(const LatentDims &d) { return d.dim + d.rot <= 256; }
 
 int latent_store_launch(const LatentDims &d, const float *proj, int64_t ldp, int M, int off_down, const float *norm_w,
                         float eps, const float *inv_freq, void *pool, const CacheView &cv, cudaStream_t st) {
-  latent_store_kernel<<<(M + 7) / 8, 256, 0, st>>>(proj, ldp, M, off_down, d, norm_w, eps, inv_freq, (bf16 *)pool, cv);
+  latent_store_kernel<<<M, 128, 0, st>>>(proj, ldp, off_down, d, norm_w, eps, inv_freq, (bf16 *)pool, cv);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

@@ -29,21 +29,41 @@ __global__ void place_rows_kernel(const S *src, int cols, D *dst, int64_t ld, in
 }
 
 template <typename T>
-__global__ void embed_table_kernel(const T *table, int64_t ld, const int32_t *tokens, float *x, int H) {
+__global__ void __launch_bounds__(256)
+embed_table_kernel(const T *table, int64_t ld, const int32_t *tokens, float *x, int H) {
+  constexpr int E = RowUnit<T>::E;
   const T *src = table + (int64_t)tokens[blockIdx.x] * ld;
-  for (int i = threadIdx.x; i < H; i += blockDim.x)
-    x[(int64_t)blockIdx.x * H + i] = to_float(src[i]);
+  float *dst = x + (int64_t)blockIdx.x * H;
+  for (int k = threadIdx.x * E; k < H; k += 256 * E) {   // rows are padded to whole units
+    const uint4 u = *reinterpret_cast<const uint4 *>(src + k);
+#pragma unroll
+    for (int g = 0; g < RowUnit<T>::NG; ++g) {
+      float f[4];
+      RowUnit<T>::group(u, g, f);
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (k + 4 * g + e < H)
+          dst[k + 4 * g + e] = f[e];
+    }
+  }
 }
 
-// h = RMSNorm(x[rows ? rows[m] : m]) as bf16 rows of ldh (zero beyond H): a CTA per row
+// h = RMSNorm(x) as bf16 rows of ldh (zero beyond H): a CTA per row
 __global__ void __launch_bounds__(256)
-norm_rows_kernel(const float *x, const int32_t *rows, int H, const float *norm_w, float eps, bf16 *h, int64_t ldh) {
+norm_rows_kernel(const float *x, int H, const float *norm_w, float eps, bf16 *h, int64_t ldh) {
   __shared__ float s_red[8];
   const int m = blockIdx.x;
-  const float *src = x + (int64_t)(rows ? rows[m] : m) * H;
+  const float *src = x + (int64_t)m * H;
+  const bool vec = (H & 3) == 0;
   float s = 0.f;
-  for (int k = threadIdx.x; k < H; k += 256)
-    s = fmaf(src[k], src[k], s);
+  if (vec)
+    for (int k = threadIdx.x * 4; k < H; k += 1024) {
+      const float4 v = *reinterpret_cast<const float4 *>(src + k);
+      s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+    }
+  else
+    for (int k = threadIdx.x; k < H; k += 256)
+      s = fmaf(src[k], src[k], s);
   s = warp_sum(s);
   if ((threadIdx.x & 31) == 0)
     s_red[threadIdx.x >> 5] = s;
@@ -52,13 +72,28 @@ norm_rows_kernel(const float *x, const int32_t *rows, int H, const float *norm_w
   for (int w = 0; w < 8; ++w)
     t += s_red[w];
   const float r = 1.0f / sqrtf(t / (float)H + eps);
-  for (int k = threadIdx.x; k < ldh; k += 256)
-    h[(int64_t)m * ldh + k] = __float2bfloat16_rn(k < H ? src[k] * r * norm_w[k] : 0.f);
+  bf16 *dst = h + (int64_t)m * ldh;
+  if (vec) {
+    for (int k = threadIdx.x * 4; k < ldh; k += 1024) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f), w = v;
+      if (k < H) {
+        v = *reinterpret_cast<const float4 *>(src + k);
+        w = __ldg(reinterpret_cast<const float4 *>(norm_w + k));
+      }
+      const __nv_bfloat162 a = __floats2bfloat162_rn(v.x * r * w.x, v.y * r * w.y), b = __floats2bfloat162_rn(v.z * r * w.z, v.w * r * w.w);
+      *reinterpret_cast<uint2 *>(dst + k) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+    }
+  } else {
+    for (int k = threadIdx.x; k < ldh; k += 256)
+      dst[k] = __float2bfloat16_rn(k < H ? src[k] * r * norm_w[k] : 0.f);
+  }
 }
 
-__global__ void gather_rows_kernel(const float *x, const int32_t *rows, float *y, int H) {
+__global__ void __launch_bounds__(256)
+gather_rows_kernel(const float *x, const int32_t *rows, float *y, int H) {
   const float *src = x + (int64_t)rows[blockIdx.x] * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x)
+#pragma unroll 4
+  for (int i = threadIdx.x; i < H; i += 256)
     y[(int64_t)blockIdx.x * H + i] = src[i];
 }
 
@@ -250,9 +285,9 @@ int reserve(b200_model *m, LayeredWs &ws, int rows, int ctx) {
   return B200_OK;
 }
 
-int norm_rows_launch(const float *x, const int32_t *rows, int H, int M, const float *norm_w, float eps, bf16 *h, int64_t ldh,
+int norm_rows_launch(const float *x, int H, int M, const float *norm_w, float eps, bf16 *h, int64_t ldh,
                      cudaStream_t st) {
-  norm_rows_kernel<<<M, 256, 0, st>>>(x, rows, H, norm_w, eps, h, ldh);
+  norm_rows_kernel<<<M, 256, 0, st>>>(x, H, norm_w, eps, h, ldh);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -274,7 +309,7 @@ int row_layers(b200_model *m, LayeredWs &ws, float *x, int M, const CacheView &c
       return rc;
     const int splits = latent_splits(L.d, M, max_ctx);
     if (int rc = latent_attend_launch(s->dtype, L.d, ws.qabs, M, pool, cv, splits, max_ctx, ws.part, st)) return rc;
-    if (int rc = latent_value_launch(s->dtype, L.d, ws.part, M, splits, L.uv, ws.cat, s->ldc, false, st)) return rc;
+    if (int rc = latent_value_launch(s->dtype, L.d, ws.part, M, splits, L.uv, ws.cat, s->ldc, false, nullptr, st)) return rc;
     if (c.ff_kind == B200_FF_EXPERTS) {
       if (int rc = expert_rows_launch(s->dtype, L.expert_in, L.expert_out, c.ff, c.experts, c.top, L.gate, x, W, M,
                                       L.norm, eps, ws.proj + L.off_router, s->ldp, &L.out, ws.cat, s->ldc, ws.mid,
@@ -319,7 +354,7 @@ int dense_attention(b200_model *m, LayeredWs &ws, LayeredLayer &L, int M, const 
                                     false, 0, nullptr, 0.f, pool, c, st))
       return rc;
     if (int rc = latent_attend_launch(s->dtype, d, ws.qabs, n, pool, c, splits, max_ctx, ws.part, st)) return rc;
-    return latent_value_launch(s->dtype, d, ws.part, n, splits, L.uv, ws.cat16 + (int64_t)r0 * s->ldc, s->ldc, true, st);
+    return latent_value_launch(s->dtype, d, ws.part, n, splits, L.uv, ws.cat16 + (int64_t)r0 * s->ldc, s->ldc, true, ws.qabs, st);
   };
   int begin = 0;                         // first row not yet attended for
   for (const RowSegment &g : segs) {
@@ -354,7 +389,7 @@ int dense_layers(b200_model *m, LayeredWs &ws, float *x, int M, const CacheView 
   for (LayeredLayer &L : s->layers) {
     const b200_layer_config &c = L.cfg;
     void *pool = pools[L.source];
-    if (int rc = norm_rows_launch(x, nullptr, W, M, L.norm, m->cfg.eps, ws.h16, ldh, st)) return rc;
+    if (int rc = norm_rows_launch(x, W, M, L.norm, m->cfg.eps, ws.h16, ldh, st)) return rc;
     GemmBf16 in;
     in.A = ws.h16; in.lda = ldh; in.M = M; in.w = L.in; in.w.N = L.plain; in.C = ws.proj; in.ldc = s->ldp;
     if (int rc = gemm_bf16_launch(in, s->gemm_ws, st)) return rc;
@@ -402,9 +437,9 @@ int embed_tokens(b200_model *m, const int32_t *tokens, float *x, int M, cudaStre
   LayeredState *s = m->lay;
   const int W = m->cfg.hidden;
   if (s->dtype == B200_F32)
-    embed_table_kernel<float><<<M, 128, 0, st>>>((const float *)s->embed.w, s->embed.ld, tokens, x, W);
+    embed_table_kernel<float><<<M, 256, 0, st>>>((const float *)s->embed.w, s->embed.ld, tokens, x, W);
   else
-    embed_table_kernel<bf16><<<M, 128, 0, st>>>((const bf16 *)s->embed.w, s->embed.ld, tokens, x, W);
+    embed_table_kernel<bf16><<<M, 256, 0, st>>>((const bf16 *)s->embed.w, s->embed.ld, tokens, x, W);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -413,7 +448,7 @@ int head(b200_model *m, const float *x, int n, float *logits, cudaStream_t st) {
   LayeredState *s = m->lay;
   if (dense(s, n) && s->gemm_ws) {
     const int64_t ldh = pad_to(m->cfg.hidden, 8);
-    if (int rc = norm_rows_launch(x, nullptr, m->cfg.hidden, n, s->final_norm, m->cfg.eps, s->h_want, ldh, st)) return rc;
+    if (int rc = norm_rows_launch(x, m->cfg.hidden, n, s->final_norm, m->cfg.eps, s->h_want, ldh, st)) return rc;
     GemmBf16 g;
     g.A = s->h_want; g.lda = ldh; g.M = n; g.w = s->embed; g.C = logits; g.ldc = m->cfg.vocab;
     return gemm_bf16_launch(g, s->gemm_ws, st);
@@ -514,7 +549,7 @@ int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row
       local.push_back(want[k] - m0);
     if (!local.empty()) {
       B200_CUDA(cudaMemcpyAsync(s->want, local.data(), local.size() * 4, cudaMemcpyHostToDevice, st));
-      gather_rows_kernel<<<(unsigned)local.size(), 128, 0, st>>>(ws.x, s->want, s->x_want + (int64_t)done * W, W);
+      gather_rows_kernel<<<(unsigned)local.size(), 256, 0, st>>>(ws.x, s->want, s->x_want + (int64_t)done * W, W);
       B200_LAUNCH_CHECK();
       done += (int)local.size();
       B200_CUDA(cudaStreamSynchronize(st));   // `local` is reused

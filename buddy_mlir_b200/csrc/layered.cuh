@@ -92,8 +92,9 @@ int64_t latent_scratch_floats(const LatentDims &d, int M, int splits);
 int latent_splits(const LatentDims &d, int M, int max_ctx);
 int latent_attend_launch(int dtype, const LatentDims &d, const float *qabs, int M, const void *pool, const CacheView &cv,
                          int splits, int max_ctx, float *scratch, cudaStream_t st);
+// work: room for M * heads * (rank + 7) bf16 (the attended queries' own buffer will do), or null
 int latent_value_launch(int dtype, const LatentDims &d, const float *scratch, int M, int splits, const RowMatrix &uv,
-                        void *out, int64_t ldo, bool out_bf16, cudaStream_t st);
+                        void *out, int64_t ldo, bool out_bf16, void *work, cudaStream_t st);
 int latent_limits(const LatentDims &d);   // 0, or an error for sizes the kernels do not take
 
 // latent_prefill.cu: many consecutive queries of one sequence, bf16

@@ -89,35 +89,42 @@ __device__ __forceinline__ void stage_row(float4 *xs, const float *x, int n, flo
   }
 }
 // acc[r][m] += sum over k < kc of row r * staged row m; kc a multiple of E, rows readable up to kc.
+// UN blocks of every row are requested before the first is used.
 template <typename T, int MT, int R>
 __device__ __forceinline__ void dot_rows(const T *const (&row)[R], int kc, const float4 *xs, int xs_ld, int lane,
                                          float (&acc)[R][MT]) {
   using U = RowUnit<T>;
   constexpr int BLK = 32 * U::E;
-  constexpr int UN = MT * R >= 16 ? 1 : (R >= 4 ? 2 : 4);
-#pragma unroll UN
-  for (int b = 0; b < kc; b += BLK) {
-    const int k = b + lane * U::E;
-    if (k < kc) {
-      uint4 wv[R];
+  constexpr int UN = MT * R >= 16 ? 2 : (R >= 4 ? 2 : (R == 2 ? 4 : 6));
+  for (int b0 = 0; b0 < kc; b0 += BLK * UN) {
+    uint4 wv[UN][R];
+#pragma unroll
+    for (int u = 0; u < UN; ++u) {
+      const int k = b0 + u * BLK + lane * U::E;
 #pragma unroll
       for (int r = 0; r < R; ++r)
-        wv[r] = ld_stream_row(row[r] + k);
+        wv[u][r] = k < kc ? ld_stream_row(row[r] + k) : make_uint4(0, 0, 0, 0);
+    }
 #pragma unroll
-      for (int g = 0; g < U::NG; ++g) {
-        float wf[R][4];
+    for (int u = 0; u < UN; ++u) {
+      const int b = b0 + u * BLK;
+      if (b + lane * U::E < kc) {
 #pragma unroll
-        for (int r = 0; r < R; ++r)
-          U::group(wv[r], g, wf[r]);
+        for (int g = 0; g < U::NG; ++g) {
+          float wf[R][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          const float4 xv = xs[m * xs_ld + (b >> 2) + g * 32 + lane];
+          for (int r = 0; r < R; ++r)
+            U::group(wv[u][r], g, wf[r]);
 #pragma unroll
-          for (int r = 0; r < R; ++r) {
-            acc[r][m] = fmaf(xv.x, wf[r][0], acc[r][m]);
-            acc[r][m] = fmaf(xv.y, wf[r][1], acc[r][m]);
-            acc[r][m] = fmaf(xv.z, wf[r][2], acc[r][m]);
-            acc[r][m] = fmaf(xv.w, wf[r][3], acc[r][m]);
+          for (int m = 0; m < MT; ++m) {
+            const float4 xv = xs[m * xs_ld + (b >> 2) + g * 32 + lane];
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+              acc[r][m] = fmaf(xv.x, wf[r][0], acc[r][m]);
+              acc[r][m] = fmaf(xv.y, wf[r][1], acc[r][m]);
+              acc[r][m] = fmaf(xv.z, wf[r][2], acc[r][m]);
+              acc[r][m] = fmaf(xv.w, wf[r][3], acc[r][m]);
+            }
           }
         }
       }
@@ -134,6 +141,32 @@ __device__ __forceinline__ float gate_pair(const Gate &p, float g, float u) {
   g = fminf(g, p.limit);
   u = fminf(fmaxf(u, -p.limit), p.limit);
   return (g / (1.0f + expf(-p.slope * g))) * (u + p.offset);
+}
+
+// mma.sync building blocks
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void *p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+// two f32 as packed bf16 (first in the low half), and what the rounding left
+__device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t &lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
+  hi = *reinterpret_cast<const uint32_t *>(&h);
+  lo = *reinterpret_cast<const uint32_t *>(&l);
 }
 
 } // namespace b200
