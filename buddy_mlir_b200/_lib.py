@@ -10,7 +10,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libbuddy_b200_kernels.so")
 
 F32, F16, BF16 = 0, 1, 2
-W_F32, W_I8, W_U4, W_BF16 = 0, 1, 2, 3
+W_F32, W_I8, W_U4 = 0, 1, 2
 MIX_LATENT = 0
 FF_NONE, FF_GATED, FF_EXPERTS = 0, 1, 2
 

@@ -2213,6 +2213,8 @@ int b200_model_kv_overflow(b200_model *m, int position, int keep, float theta,
                            int *new_position) {
   if (!m || !new_position)
     return fail(B200_EINVAL, "model_kv_overflow: null argument");
+  if (m->lay)
+    return layered_kv_overflow(m, position, keep, new_position);
   if (int rc = b200_kv_overflow(m->kv_dev, (int)m->kv.size(), m->kvh, m->cfg.max_len,
                                 m->cfg.head_dim, position, keep, theta, new_position,
                                 m->stream))

@@ -205,5 +205,6 @@ int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row
                  const int32_t *want, float *logits_host, int32_t *next_host);
 int layered_status(b200_model *m);                      // after a synchronise: did a bounded wait give up?
 int layered_clear_cache(b200_model *m);
+int layered_kv_overflow(b200_model *m, int position, int keep, int *new_position);
 int64_t layered_step_bytes(const b200_model *m, int ctx);
 } // namespace b200

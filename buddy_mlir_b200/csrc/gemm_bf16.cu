@@ -1,6 +1,6 @@
-// bf16 x bf16 -> f32 GEMM on the 5th-generation tensor cores over plain weight rows
-// (B200_W_BF16): C[M, N] = A[M, K] * W[N, K]^T, for prefill and batched decode of models whose
-// weights are bfloat16.
+// bf16 x bf16 -> f32 GEMM on the 5th-generation tensor cores over plain weight rows,
+// C[M, N] = A[M, K] * W[N, K]^T, for prefill and batched decode of models whose weights are
+// bfloat16.
 //
 // Both operands arrive by TMA (cp.async.bulk.tensor, no multicast) as 128-byte-swizzled rows of
 // 64 k; one thread issues tcgen05.mma (128 x 128 or 128 x 256 x 16) into a f32 accumulator in

@@ -1,4 +1,4 @@
-// GEMV over plain weight rows (B200_W_F32 / B200_W_BF16), up to eight activation rows per pass:
+// GEMV over plain weight rows (f32 or bfloat16), up to eight activation rows per pass:
 //   y[m, n] (+)= sum_k norm(x)[m, k] * w[n, k]
 // with an optional RMSNorm prologue, a residual sum, and gated (gate, up) row pairs from a given
 // row on, so that one launch serves every projection that reads the same normalised row.

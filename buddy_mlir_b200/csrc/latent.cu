@@ -238,6 +238,23 @@ latent_prep_mma_kernel(const PrepP p) {
   }
 }
 
+// cache rows [src, src + tail) of one sequence -> stage, their key parts turned by `delta` positions
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_shift_kernel(const T *cache, LatentDims d, int src, const float *inv_freq, float delta, T *stage) {
+  const T *from = cache + (int64_t)(src + blockIdx.x) * d.row;
+  T *to = stage + (int64_t)blockIdx.x * d.row;
+  for (int k = threadIdx.x; k < (int)d.row; k += 128)
+    if (k < d.rank || k >= d.rank + d.rot)
+      to[k] = from[k];
+  for (int i = threadIdx.x; i < d.rot / 2; i += 128) {
+    float a, b;
+    rotate(to_float(from[d.rank + 2 * i]), to_float(from[d.rank + 2 * i + 1]), delta * inv_freq[i], a, b);
+    to[d.rank + 2 * i] = from_float<T>(a);
+    to[d.rank + 2 * i + 1] = from_float<T>(b);
+  }
+}
+
 struct AttendP {
   const float *qabs;
   const void *pool;
@@ -827,6 +844,16 @@ int latent_limits(const LatentDims &d) {
   if (d.rank > 1024 || d.rot > 256 || d.heads > 1024)
     return fail(B200_ELIMIT, "latent attention: rank %d (limit 1024), rot %d (limit 256), heads %d (limit 1024)", d.rank,
                 d.rot, d.heads);
+  return B200_OK;
+}
+
+int latent_shift_launch(int dtype, const LatentDims &d, const void *cache, int src, int tail, const float *inv_freq, int delta,
+                        void *stage, cudaStream_t st) {
+  if (dtype == B200_F32)
+    latent_shift_kernel<float><<<tail, 128, 0, st>>>((const float *)cache, d, src, inv_freq, (float)delta, (float *)stage);
+  else
+    latent_shift_kernel<bf16><<<tail, 128, 0, st>>>((const bf16 *)cache, d, src, inv_freq, (float)delta, (bf16 *)stage);
+  B200_LAUNCH_CHECK();
   return B200_OK;
 }
 

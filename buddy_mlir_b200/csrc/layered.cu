@@ -486,6 +486,41 @@ int layered_clear_cache(b200_model *m) {
   return B200_OK;
 }
 
+// The session's cache is full: keep the first `keep` positions, drop half of the rest, move what
+// remains up to them (the same choice of rows as b200_kv_overflow).
+int layered_kv_overflow(b200_model *m, int position, int keep, int *new_position) {
+  LayeredState *s = m->lay;
+  const int max_len = m->cfg.max_len;
+  if (position < max_len) {
+    *new_position = -1;
+    return B200_OK;
+  }
+  const int cur = max_len;
+  keep = std::max(0, std::min(keep, cur - 1));
+  const int discard = std::max(1, (cur - keep) / 2), src = keep + discard, tail = cur - src;
+  cudaStream_t st = m->stream;
+  void *stage = nullptr;
+  if (int rc = dev_alloc(&stage, (size_t)std::max(1, tail) * s->max_row * elem(s->dtype))) return rc;
+  int rc = B200_OK;
+  for (LayeredLayer &L : s->layers) {
+    if (!L.own() || rc)
+      continue;
+    const size_t row = (size_t)L.d.row * elem(s->dtype);
+    if (tail > 0) {
+      rc = latent_shift_launch(s->dtype, L.d, L.cache, src, tail, L.inv_freq, -discard, stage, st);
+      if (!rc && cudaMemcpyAsync((char *)L.cache + keep * row, stage, tail * row, cudaMemcpyDeviceToDevice, st) != cudaSuccess)
+        rc = fail(B200_ECUDA, "kv_overflow: moving the cache rows failed");
+    }
+    if (!rc && cudaMemsetAsync((char *)L.cache + (keep + tail) * row, 0, (cur - keep - tail) * row, st) != cudaSuccess)
+      rc = fail(B200_ECUDA, "kv_overflow: clearing the cache rows failed");
+  }
+  if (cudaStreamSynchronize(st) != cudaSuccess && !rc)
+    rc = fail(B200_ECUDA, "kv_overflow: %s", cudaGetErrorString(cudaGetLastError()));
+  cudaFree(stage);
+  *new_position = cur - discard;
+  return rc;
+}
+
 int layered_issue_step(b200_model *m, cudaStream_t st) {
   LayeredState *s = m->lay;
   if (int rc = reserve(m, s->one, 1, m->cfg.max_len)) return rc;

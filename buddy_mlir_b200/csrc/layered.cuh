@@ -95,6 +95,8 @@ int latent_attend_launch(int dtype, const LatentDims &d, const float *qabs, int 
 // work: room for M * heads * (rank + 7) bf16 (the attended queries' own buffer will do), or null
 int latent_value_launch(int dtype, const LatentDims &d, const float *scratch, int M, int splits, const RowMatrix &uv,
                         void *out, int64_t ldo, bool out_bf16, void *work, cudaStream_t st);
+int latent_shift_launch(int dtype, const LatentDims &d, const void *cache, int src, int tail, const float *inv_freq, int delta,
+                        void *stage, cudaStream_t st);   // rows moved by `delta` positions, into stage
 int latent_limits(const LatentDims &d);   // 0, or an error for sizes the kernels do not take
 
 // latent_prefill.cu: many consecutive queries of one sequence, bf16

@@ -1,4 +1,4 @@
-// Plain weight rows (B200_W_F32 and B200_W_BF16 keep k in its natural order): the streaming dot
+// Plain weight rows (f32 or bfloat16, k in its natural order): the streaming dot
 // product that the GEMV-shaped kernels share, and the gate of a gated feed-forward pair.
 #pragma once
 #include "common.cuh"

@@ -53,8 +53,7 @@ enum { B200_F32 = 0, B200_F16 = 1, B200_BF16 = 2 };
 enum {
   B200_W_F32 = 0, /* f32, row n = output channel, K contiguous            */
   B200_W_I8 = 1,  /* int8, per-output-channel scale                       */
-  B200_W_U4 = 2,  /* 4-bit, value = nibble - 8, one scale per `group` k    */
-  B200_W_BF16 = 3 /* bfloat16, row n = output channel, K contiguous        */
+  B200_W_U4 = 2   /* 4-bit, value = nibble - 8, one scale per `group` k    */
 };
 
 /* ------------------------------------------------------------------------
@@ -472,7 +471,9 @@ int b200_model_tp_sum_kind(const b200_model *m);
 int b200_model_read_trace(b200_model *m, long long *host, int64_t capacity);
 /* Session handle -> device pointers, for tests. */
 float *b200_model_kv_ptr(b200_model *m, int buffer);
-/* KV overflow on the device-resident cache; see b200_kv_overflow. */
+/* KV overflow on the device-resident cache; see b200_kv_overflow.  Models of
+ * described layers: the cached rows move the same way and their rotated key
+ * parts are turned back by the layer's own rotation (theta is not read). */
 int b200_model_kv_overflow(b200_model *m, int position, int keep, float theta,
                            int *new_position);
 

@@ -351,6 +351,28 @@ def test_greedy_generation_and_device_loop():
     s.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_full_cache_drops_positions_and_turns_keys_back(dtype):
+    """One layer: its cached rows depend on nothing but token and position, so after the overflow
+    the session must continue like a fresh sequence of the tokens that were kept."""
+    cfg = tz.config([(tz.attention(window=30), tz.gated())])
+    w = tz.weights(cfg, 31)
+    s = tz.session(cfg, w, dtype, max_len=48)
+    toks = tokens(cfg, 48, 3)
+    s.prefill_rows(toks, 0)
+    assert not tz.session(cfg, w, dtype, max_len=60).handle_kv_cache_overflow(4)
+    assert s.handle_kv_cache_overflow(10)
+    kept = np.concatenate([toks[:10], toks[29:]])
+    assert s.position() == len(kept)
+    for t in (5, 6, 7):
+        kept = np.append(kept, t)
+        s.decode(t)
+        assert tz.error(s.logits_data(), tz.want_logits(cfg, w, kept)[-1]) < tz.TOLERANCE[dtype]
+    ids, _ = run_generation(s, [int(t) for t in toks[:40]], 40 + 30)   # runs past the cache's end
+    assert len(ids) == 31
+    s.close()
+
+
 def test_batched_greedy_generation():
     cfg, w = tz.mixed_model(22)
     s = tz.session(cfg, w, "float32")
