@@ -87,6 +87,15 @@ def route(h, router, top):
     return chosen, e / e.sum(axis=-1, keepdims=True)
 
 
+def route_margin(h, router, top):
+    """How far the last chosen expert's logit lies above the first one left out, per token, relative
+    to the spread of the logits: a small margin may fall either way under rounding."""
+    z = np.sort(h @ router.T, axis=-1)[:, ::-1]
+    if top == z.shape[1]:
+        return np.full(len(h), np.inf)
+    return (z[:, top - 1] - z[:, top]) / z.std()
+
+
 def mixture(h, mlp, tensors, prefix):
     limit = mlp["expert"]["limit"]
     chosen, weight = route(h, tensors[prefix + "router"], mlp["router"]["top"])
@@ -104,9 +113,9 @@ def feed_forward(h, mlp, tensors, prefix):
     return mixture(h, mlp, tensors, prefix)
 
 
-def forward(config, tensors, tokens, dtype=np.float64, residuals=None):
+def forward(config, tensors, tokens, dtype=np.float64, residuals=None, margins=None):
     """Logits [tokens, vocab] of one sequence; residuals (a list) receives the stream after
-    every layer."""
+    every layer, margins (a list) route_margin of every mixture."""
     t = {k: np.asarray(v).astype(dtype) for k, v in tensors.items()}
     eps = config["norm"]["eps"]
     x = t["embed"][np.asarray(tokens)]
@@ -120,6 +129,8 @@ def forward(config, tensors, tokens, dtype=np.float64, residuals=None):
             caches[i] = latent_keys(h, mixer, t, p + "mix.", eps)
             source = i
         y = latent_attention(h, *caches[source], mixer, t, p + "mix.")
+        if margins is not None and layer["mlp"] is not None and layer["mlp"]["kind"] != "dense":
+            margins.append(route_margin(h, t[p + "mlp.router"], layer["mlp"]["router"]["top"]))
         if layer["mlp"] is not None:
             y = y + feed_forward(h, layer["mlp"], t, p + "mlp.")
         x = x + y

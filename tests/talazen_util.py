@@ -68,6 +68,15 @@ def want_logits(cfg, w, tokens):
     return plain.forward(cfg, values(w), tokens)
 
 
+def clear_of_close_calls(cfg, w, tokens, margin=0.03):
+    """Per token: no router had to make a close call, which bfloat16 rounding may turn, for it or for
+    any token before it (what a token sees)."""
+    margins = []
+    plain.forward(cfg, values(w), tokens, margins=margins)
+    worst = np.min(margins, axis=0) if margins else np.full(len(tokens), np.inf)
+    return np.minimum.accumulate(worst) > margin
+
+
 def error(got, want):
     """Largest row error: rms over the vocabulary of the difference (mean taken off), relative to
     the rms of the wanted logits."""

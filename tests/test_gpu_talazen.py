@@ -8,6 +8,7 @@ import sys
 import numpy as np
 import pytest
 
+import plain_talazen as plain
 import talazen_util as tz
 from buddy_mlir_b200 import _lib
 from buddy_mlir_b200.session import run_generation
@@ -105,6 +106,50 @@ def test_shared_cache_has_its_own_heads_and_window(dtype):
     s.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_odd_sizes_everywhere(dtype):
+    cfg = tz.config([(tz.attention(heads=3, dim=7, rot=2, vdim=5, rank=11, window=13), tz.gated(ff=13)),
+                     (tz.attention(heads=1, dim=9, rot=6, vdim=3, rank=21, window=4), tz.experts(n=3, top=1, ff=7)),
+                     (tz.attention(heads=5, dim=3, rot=2, vdim=1, rank=11, kv_from=0, window=50), tz.experts(n=3, top=3, ff=9))],
+                    width=75, vocab=131)
+    w = tz.weights(cfg, 14)
+    toks = tokens(cfg, 80, 1)
+    want = tz.want_logits(cfg, w, toks)
+    s = tz.session(cfg, w, dtype)
+    assert tz.error(s.prefill_rows(toks, 0), want) < tz.TOLERANCE[dtype]
+    b = tz.batch(s)
+    assert tz.error(step_logits(b, b.add(), toks, [40, 1, 1, 10, 3, 25]), want) < tz.TOLERANCE[dtype]
+    b.close()
+    s.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_wide_projections(dtype):
+    """Large enough for every form of the contractions: 256-column tiles, a split k range, activations
+    staged in several pieces, grouped tiles of many experts."""
+    cfg = tz.config([(tz.attention(heads=6, dim=64, rot=32, vdim=64, rank=128, window=90, sharp=1.0), tz.gated(ff=4100)),
+                     (tz.attention(heads=6, dim=64, rot=32, vdim=64, rank=128, window=300, sharp=1.0), tz.experts(n=40, top=2, ff=520))],
+                    width=1032, vocab=1000)
+    w = tz.weights(cfg, 15)
+    toks = tokens(cfg, 600, 1)
+    margins = []
+    want = plain.forward(cfg, tz.values(w), toks, margins=margins)
+    clear = margins[0] > 0.03                # a close call of the router may fall either way in bfloat16
+    assert clear.mean() > 0.8
+    s = tz.session(cfg, w, dtype, max_len=640)
+    got = s.prefill_rows(toks, 0)
+    assert tz.error(got[clear], want[clear]) < tz.TOLERANCE[dtype]
+    s.reset_position()
+    s.prefill_rows(toks[:500], 0)
+    part = s.prefill_rows(toks[500:530], 500)
+    assert tz.error(part[clear[500:530]], want[500:530][clear[500:530]]) < tz.TOLERANCE[dtype]
+    for i in range(530, 538):
+        s.decode(int(toks[i]))
+        if clear[i]:
+            assert tz.error(s.logits_data(), want[i]) < tz.TOLERANCE[dtype]
+    s.close()
+
+
 # ---- the whole model under schedules -----------------------------------------------------------
 @pytest.fixture(scope="module", params=DTYPES)
 def mixed(request):
@@ -116,7 +161,7 @@ def mixed(request):
 
 
 @pytest.mark.parametrize("page", [1, 4, 16, 100])
-@pytest.mark.parametrize("size", [2, 3, 8, 9, 17, 50, 200])
+@pytest.mark.parametrize("size", [2, 3, 8, 9, 16, 17, 50, 200])
 def test_portions(mixed, size, page):
     cfg, w, s, toks, want, tol = mixed
     n = 60 if size < 8 else len(toks)
@@ -202,6 +247,23 @@ def test_unequal_batch_against_each_alone(mixed):
             got, nxt = b.step(entries, want_places)
             assert tz.error(got, np.array(expect)) < tol
             assert np.array_equal(nxt, got.argmax(axis=1))
+    b.close()
+
+
+def test_many_sequences_in_one_step(mixed):
+    cfg, w, s, _, _, tol = mixed
+    rng = np.random.default_rng(17)
+    seqs = [rng.integers(0, cfg["vocab"], 5 + i % 4) for i in range(70)]
+    b = tz.batch(s, max_seqs=70, page=4)
+    ids = [b.add() for _ in seqs]
+    b.step([(q, t[:-3]) for q, t in zip(ids, seqs)])
+    got = [b.step([(q, t[k:k + 1] if k < -1 else t[-1:]) for q, t in zip(ids, seqs)])[0] for k in (-3, -2, -1)]
+    compared = 0
+    for i, t in enumerate(seqs):
+        if tol < 1e-3 or tz.clear_of_close_calls(cfg, w, t)[-1]:
+            compared += 1
+            assert tz.error(np.array([g[i] for g in got]), tz.want_logits(cfg, w, t)[-3:]) < tol
+    assert compared > 20
     b.close()
 
 
