@@ -3,6 +3,7 @@
 
     python bench.py --gpus 1 --steps 256 --warmup 8
     python bench.py --impl reference --steps 64 --warmup 3
+    python bench.py --layered        # models of described layers beside the uniform one
 
 N = 1 workload (the configuration the headline metric is quoted on): the
 DeepSeek-R1-Distill-Qwen-1.5B architecture with int8 per-output-channel
@@ -629,6 +630,8 @@ def run_layered_only(args):
         raise SystemExit("bench.py needs a CUDA device; the library has no CPU path")
     torch.cuda.set_device(0)
     out = {}
+    sampler = ClockSampler(0)
+    sampler.start()
     for name in ([args.layered_shape] if args.layered_shape else LAYERED_SHAPES):
         out[name] = {}
         for kind, make in (("talazen_bf16", layered_model), ("uniform_int8", uniform_model)):
@@ -637,7 +640,8 @@ def run_layered_only(args):
             s = make(name)
             out[name][kind] = session_numbers(s)
             s.close()
-    print(json.dumps({"layered": out, "sizes": LAYERED,
+    print(json.dumps({"layered": out, "sizes": LAYERED, "clocks": sampler.stop(),
+                      "l2": "weights of a step larger than L2",
                       "shapes": {k: dict(zip(("hidden", "heads", "kv_heads_uniform", "ff_dense_or_active", "experts", "top", "expert_ff"), v))
                                  for k, v in LAYERED_SHAPES.items()}, "data": "synthetic, seeded weights"}))
 

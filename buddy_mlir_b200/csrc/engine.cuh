@@ -79,7 +79,7 @@ struct LayeredTensor {         // where a named tensor goes
   bool set;
 };
 struct LayeredWs {             // activations of up to `rows` rows
-  int rows = 0, ctx = 0, part_rows = 0;
+  int rows = 0, ctx = 0;
   std::vector<void *> owned;
   float *proj = nullptr, *qabs = nullptr, *part = nullptr, *cat = nullptr, *mid = nullptr, *weight = nullptr;
   int32_t *ids = nullptr;
@@ -98,7 +98,7 @@ struct LayeredState {
   std::map<std::string, LayeredTensor> tensors;
   std::vector<void *> owned;
   int32_t *zero = nullptr;     // sequence 0, page 0: the session's block table
-  int ldp = 0, ldc = 0, ldq = 0, max_mid = 0, max_slots = 0, max_ff = 0, max_top = 0, max_experts = 0;
+  int ldp = 0, ldc = 0, ldq = 0, max_mid = 0, max_ff = 0, max_top = 0, max_experts = 0;
   int max_q = 0, max_row = 0, max_kv = 0;
   int window = 0;              // the widest window of all layers, 0: some layer sees everything
   LayeredWs one, many;         // the captured decode step's rows, and everything else's

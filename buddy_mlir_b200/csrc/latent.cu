@@ -304,7 +304,7 @@ latent_attend_kernel(const AttendP p) {
   for (int kb = k0; kb < k1; kb += kKeys) {
     const int nk = min(kKeys, k1 - kb);
     __syncthreads();
-    // a warp brings in the tile's rows 4 apart..: rows of one page are contiguous
+    // a warp brings in every eighth row of the tile
     for (int r = warp; r < nk; r += 8) {
       const T *src = reinterpret_cast<const T *>(p.pool) + cache_row(p.cv, seq, kb + r) * d.row;
       for (int u = lane; u < units; u += 32)

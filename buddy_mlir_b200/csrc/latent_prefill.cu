@@ -111,7 +111,7 @@ struct FlashP {
   const bf16 *rows;            // [keys][row]: cache rows from position `first` on
   const bf16 *kv;              // [keys][ldkv]: heads * dim keys, then heads * vdim values
   int64_t ldkv;
-  int first, n_keys;
+  int first;
   bf16 *out;                   // [n][ldo]
   int64_t ldo;
   LatentDims d;
@@ -358,7 +358,7 @@ int latent_prefill_launch(const LatentDims &d, const bf16 *q, int n, int pos0, c
                           int first, bf16 *out, int64_t ldo, cudaStream_t st) {
   FlashP p{};
   p.q = q; p.n = n; p.pos0 = pos0; p.rows = rows; p.kv = kv; p.ldkv = ldkv; p.first = first;
-  p.n_keys = pos0 + n - first; p.out = out; p.ldo = ldo; p.d = d;
+  p.out = out; p.ldo = ldo; p.d = d;
   p.vec = d.dim % 8 == 0 && d.rot % 8 == 0 && d.vdim % 8 == 0 && d.rank % 8 == 0 && ldkv % 8 == 0;
   const int dk = d.dim + d.rot;
   if (dk <= 64) return flash_values<64>(p, st);

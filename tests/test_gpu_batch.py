@@ -116,3 +116,30 @@ def test_batch_limits_are_reported():
         bs.decode([a, a], [1, 2])                  # a sequence listed twice
     bs.close()
     s.close()
+
+
+def test_mixed_step_matches_per_sequence_checker():
+    """Prompts and single tokens in one step, logits asked for at scattered places."""
+    cfg = TINY_QWEN2
+    _, views = synthetic.make_f32_blob(cfg, 62)
+    s = ModelSession(cfg)
+    s.load_tensors(views)
+    bs = BatchSession(s, max_seqs=3, page_size=8, n_pages=30, max_context=cfg.max_len)
+    rng = np.random.default_rng(4)
+    seqs = [rng.integers(0, cfg.vocab, n) for n in (20, 9, 14)]
+    wants = []
+    for t in seqs:
+        om = orc.OracleModel(cfg, views)
+        wants.append(np.array([om.decode(int(x)).copy() for x in t]))
+    ids = [bs.add() for _ in seqs]
+    got, _ = bs.step([(ids[0], seqs[0][:12]), (ids[1], seqs[1][:1])], [[11, 3], []])
+    assert maxrel(got, wants[0][[11, 3]]) < 1e-3
+    got, nxt = bs.step([(ids[1], seqs[1][1:]), (ids[0], seqs[0][12:13]), (ids[2], seqs[2])], [[0, 7], [0], [13, 0]])
+    want = np.array([wants[1][1], wants[1][8], wants[0][12], wants[2][13], wants[2][0]])
+    assert maxrel(got, want) < 1e-3
+    assert nxt.tolist() == [greedy_sample(w) for w in want]
+    bs.step([(ids[0], seqs[0][13:19])], [[]])
+    got, _ = bs.step([(ids[0], seqs[0][19:])])
+    assert maxrel(got, wants[0][[19]]) < 1e-3
+    bs.close()
+    s.close()
