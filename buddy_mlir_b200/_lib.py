@@ -11,8 +11,10 @@ LIB_PATH = os.path.join(_HERE, "libbuddy_b200_kernels.so")
 
 F32, F16, BF16 = 0, 1, 2
 W_F32, W_I8, W_U4 = 0, 1, 2
-MIX_LATENT = 0
-FF_NONE, FF_GATED, FF_EXPERTS = 0, 1, 2
+MIX_LATENT, MIX_HEADS, MIX_MEMORY, MIX_HEADS_MEMORY = 0, 1, 2, 3
+BLOCK_PARALLEL, BLOCK_SANDWICH = 0, 1
+FF_NONE, FF_GATED, FF_EXPERTS, FF_PLAIN = 0, 1, 2, 3
+ACT_NONE, ACT_RELU2, ACT_GELU_TANH = 0, 1, 2
 
 (T_EMBED, T_INV_FREQ, T_FINAL_NORM, T_LM_HEAD, T_IN_NORM, T_POST_NORM, T_Q_NORM,
  T_K_NORM, T_Q, T_K, T_V, T_O, T_GATE, T_UP, T_DOWN, T_Q_BIAS, T_K_BIAS,
@@ -61,7 +63,16 @@ class LayerConfigC(C.Structure):
                 ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "kv_from")] + \
                [("scale", C.c_float), ("rot_base", C.c_float)] + \
                [(n, C.c_int32) for n in ("ff_kind", "ff", "experts", "top")] + \
-               [(n, C.c_float) for n in ("limit", "gate_slope", "up_offset")]
+               [(n, C.c_float) for n in ("limit", "gate_slope", "up_offset")] + \
+               [(n, C.c_int32) for n in ("block", "ff_act", "kv_heads", "rot_halves", "qkv_bias", "qk_norm", "out_gate")] + \
+               [(n, C.c_float) for n in ("sink", "mix_scale")] + \
+               [(n, C.c_int32) for n in ("mem_heads", "mem_dim", "mem_vdim")] + \
+               [(n, C.c_float) for n in ("mem_cap", "mem_q_scale", "mem_floor", "mem_mix_scale")]
+
+
+class StackConfigC(C.Structure):
+    _fields_ = [("embed_scale", C.c_float)] + \
+               [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "side_dim")]
 
 
 class B200Error(RuntimeError):
@@ -116,7 +127,8 @@ def load():
         "b200_kv_overflow": (i32, [vp, i32, i32, i32, i32, i32, i32, f32,
                                    C.POINTER(C.c_int), vp]),
         "b200_model_create": (i32, [C.POINTER(ModelConfigC), C.POINTER(vp)]),
-        "b200_model_create_layered": (i32, [C.POINTER(ModelConfigC), C.POINTER(LayerConfigC), i32, C.POINTER(vp)]),
+        "b200_model_create_layered": (i32, [C.POINTER(ModelConfigC), C.POINTER(StackConfigC),
+                                            C.POINTER(LayerConfigC), i32, C.POINTER(vp)]),
         "b200_model_set_tensor": (i32, [vp, C.c_char_p, i32, vp, i64, i64]),
         "b200_model_read_residual": (i32, [vp, vp, i32]),
         "b200_model_destroy": (None, [vp]),

@@ -5,11 +5,12 @@ ModelConfig: the shapes of the decode path (the configs buddy-mlir's specs bake 
 its generated ModelSession: tools/buddy-codegen/gen_session.py:156-180,
 models/deepseek_r1/specs/*.json)."""
 import ctypes as C
+import math
 from dataclasses import dataclass, replace
-from typing import Optional, Tuple
+from typing import Optional, Tuple, Union
 
 from . import _lib
-from ._lib import LayerConfigC, ModelConfigC
+from ._lib import LayerConfigC, ModelConfigC, StackConfigC
 
 
 @dataclass(frozen=True)
@@ -66,6 +67,46 @@ class LatentMixer:
 
 
 @dataclass(frozen=True)
+class HeadsMixer:
+    """Attention over keys and values cached per key/value head, with rotary positions on the first
+    rot_dim dimensions of a head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot_dim: int
+    rot_base: float
+    scale: float
+    rot_halves: bool = False         # pairs (i, i + rot_dim/2); else (2i, 2i + 1)
+    bias: bool = False               # on the query, key and value projections
+    qk_norm: bool = False            # RMSNorm over the whole query and the whole key projection
+    sink: float = -math.inf          # score of one more softmax entry that has no value
+    out_gate: bool = False           # heads times sigmoid(W_g h)
+    window: int = 0                  # 0: every position before
+
+
+@dataclass(frozen=True)
+class MemoryMixer:
+    """Matrix memory: a gated recurrent [dim][vdim] state per head, with soft-capped exponential
+    gates, a normaliser and a running maximum."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    q_scale: float
+    floor: float                     # added to the normaliser
+
+
+@dataclass(frozen=True)
+class SideBySide:
+    """Two mixers on the same input; the sum of their outputs, each times its factor."""
+    left: HeadsMixer
+    right: MemoryMixer
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass(frozen=True)
 class GatedFF:
     """down(g * sigmoid(gate_slope * g) * (u + up_offset)), g <= limit, |u| <= limit.  With
     experts > 0 a router picks `top` of that many such units per token, weighted by the softmax
@@ -79,23 +120,59 @@ class GatedFF:
 
 
 @dataclass(frozen=True)
+class PlainFF:
+    """down(act(up h)), act one of _lib.ACT_*."""
+    ff: int
+    act: int
+
+
+def _heads_fields(m, scale=1.0):
+    return dict(heads=m.heads, kv_heads=m.kv_heads, dim=m.dim, vdim=m.vdim, rot_dim=m.rot_dim, rot_base=m.rot_base,
+                scale=m.scale, rot_halves=int(m.rot_halves), qkv_bias=int(m.bias), qk_norm=int(m.qk_norm),
+                out_gate=int(m.out_gate), sink=m.sink, window=m.window, mix_scale=scale)
+
+
+def _memory_fields(m, scale=1.0):
+    return dict(mem_heads=m.heads, mem_dim=m.dim, mem_vdim=m.vdim, mem_cap=m.gate_cap, mem_q_scale=m.q_scale,
+                mem_floor=m.floor, mem_mix_scale=scale)
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentMixer
-    ff: Optional[GatedFF]
+    """A mixer and a feed-forward.  Latent mixers run as a parallel block, x += mixer(h) + ff(h) with
+    h = RMSNorm(x); the others as a sandwich, x += norm1b(mixer(norm1(x))), x += norm2b(ff(norm2(x)))."""
+    mixer: Union[LatentMixer, HeadsMixer, MemoryMixer, SideBySide]
+    ff: Union[GatedFF, PlainFF, None]
 
     def to_c(self):
         m, f = self.mixer, self.ff
-        kind = _lib.FF_NONE if f is None else (_lib.FF_EXPERTS if f.experts else _lib.FF_GATED)
-        return LayerConfigC(_lib.MIX_LATENT, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.window,
-                            -1 if m.kv_from is None else m.kv_from, m.scale, m.rot_base, kind,
-                            f.ff if f else 0, f.experts if f else 0, f.top if f else 0,
-                            f.limit if f else 0.0, f.gate_slope if f else 0.0, f.up_offset if f else 0.0)
+        c = dict(kv_from=-1, mix_scale=1.0, mem_mix_scale=1.0, sink=-math.inf)
+        if isinstance(m, LatentMixer):
+            c.update(mixer=_lib.MIX_LATENT, block=_lib.BLOCK_PARALLEL, heads=m.heads, dim=m.dim, rot_dim=m.rot_dim,
+                     vdim=m.vdim, kv_rank=m.kv_rank, window=m.window, kv_from=-1 if m.kv_from is None else m.kv_from,
+                     scale=m.scale, rot_base=m.rot_base)
+        else:
+            c.update(block=_lib.BLOCK_SANDWICH)
+            if isinstance(m, HeadsMixer):
+                c.update(_heads_fields(m), mixer=_lib.MIX_HEADS)
+            elif isinstance(m, MemoryMixer):
+                c.update(_memory_fields(m), mixer=_lib.MIX_MEMORY)
+            else:
+                c.update(_heads_fields(m.left, m.left_scale), **_memory_fields(m.right, m.right_scale),
+                         mixer=_lib.MIX_HEADS_MEMORY)
+        if f is None:
+            c.update(ff_kind=_lib.FF_NONE)
+        elif isinstance(f, PlainFF):
+            c.update(ff_kind=_lib.FF_PLAIN, ff=f.ff, ff_act=f.act)
+        else:
+            c.update(ff_kind=_lib.FF_EXPERTS if f.experts else _lib.FF_GATED, ff=f.ff, experts=f.experts, top=f.top,
+                     limit=f.limit, gate_slope=f.gate_slope, up_offset=f.up_offset)
+        return LayerConfigC(**c)
 
 
 @dataclass(frozen=True)
 class LayeredConfig:
-    """A model of described layers: parallel blocks x += mixer(h) + ff(h), h = RMSNorm(x), and the
-    transposed embedding table as the output head."""
+    """A model of described layers, with the transposed embedding table as the output head."""
     name: str
     hidden: int
     vocab: int
@@ -103,6 +180,10 @@ class LayeredConfig:
     layers: Tuple[LayerSpec, ...]
     max_len: int = 4096              # positions of a single-sequence session's cache
     dtype: str = "bfloat16"          # or "float32"
+    embed_scale: float = 1.0         # factor on the embedding rows (not on the head)
+    loop: Tuple[int, int, int] = (0, 0, 1)   # layers start .. stop-1 run `times` times, with a cache per pass;
+                                     # the embedding output is added before every pass but the first
+    side_dim: int = 0                # per-token layer input of that size (sandwich layers), 0: none
 
     @property
     def n_layers(self):
@@ -112,9 +193,10 @@ class LayeredConfig:
         """b200_model_create_layered into `handle`."""
         c = ModelConfigC(hidden=self.hidden, n_layers=self.n_layers, vocab=self.vocab, max_len=self.max_len,
                          eps=self.eps, tp_rank=tp_rank, tp_size=tp_size)
+        stack = StackConfigC(self.embed_scale, *self.loop, self.side_dim)
         arr = (LayerConfigC * self.n_layers)(*[l.to_c() for l in self.layers])
         dtype = {"bfloat16": _lib.BF16, "float32": _lib.F32}[self.dtype]
-        return lib.b200_model_create_layered(C.byref(c), arr, dtype, C.byref(handle))
+        return lib.b200_model_create_layered(C.byref(c), C.byref(stack), arr, dtype, C.byref(handle))
 
     def with_(self, **kw):
         return replace(self, **kw)

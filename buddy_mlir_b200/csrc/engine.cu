@@ -1626,6 +1626,8 @@ int b200_model_decode(b200_model *m, int token, int pos, float *logits_host,
     return fail(B200_ESTATE, "decode: call b200_model_finalize first");
   if (token < 0 || token >= m->cfg.vocab || pos < 0 || pos >= m->cfg.max_len)
     return fail(B200_EINVAL, "decode: token %d / position %d out of range", token, pos);
+  if (m->lay)
+    if (int rc = layered_state_enter(m, pos)) return rc;
   if (int rc = set_state(m, token, pos)) return rc;
   B200_CUDA(cudaEventRecord(m->ev0, m->stream));
   if (int rc = run_step(m)) return rc;
@@ -1646,6 +1648,8 @@ int b200_model_decode(b200_model *m, int token, int pos, float *logits_host,
   B200_CUDA(cudaStreamSynchronize(m->stream));
   B200_CUDA(cudaEventElapsedTime(&m->last_ms, m->ev0, m->ev1));
   if (int rc = check_step_error(m)) return rc;
+  if (m->lay)
+    layered_state_leave(m, pos + 1);
   if (logits_host) {
     memcpy(logits_host, m->h_logits_pinned, (size_t)m->cfg.vocab * 4);
     m->rows_fresh = true;
@@ -1666,6 +1670,8 @@ int b200_model_generate(b200_model *m, int token, int pos, int steps,
     return fail(B200_EINVAL, "generate: %d steps from position %d exceed max_len %d",
                 steps, pos, m->cfg.max_len);
   m->rows_fresh = false;
+  if (m->lay)
+    if (int rc = layered_state_enter(m, pos)) return rc;
   if (int rc = set_state(m, token, pos)) return rc;
   B200_CUDA(cudaEventRecord(m->ev0, m->stream));
   for (int s = 0; s < steps; ++s)
@@ -1676,7 +1682,10 @@ int b200_model_generate(b200_model *m, int token, int pos, int steps,
   B200_CUDA(cudaMemcpyAsync(m->h_state_pinned, m->d_state, 32, cudaMemcpyDeviceToHost, m->stream));
   B200_CUDA(cudaStreamSynchronize(m->stream));
   B200_CUDA(cudaEventElapsedTime(&m->last_ms, m->ev0, m->ev1));
-  return check_step_error(m);
+  if (int rc = check_step_error(m)) return rc;
+  if (m->lay)
+    layered_state_leave(m, pos + steps);
+  return B200_OK;
 }
 
 // A W8A8 projection over M rows (QuantizedMatmulOp / QuantizedAddMMOp of the w8a8 graphs,
@@ -1782,25 +1791,19 @@ int b200_model_prefill(b200_model *m, const int32_t *tokens, int n_tokens, int p
       return fail(B200_EINVAL, "prefill: token %d at row %d out of range", tokens[i], i);
   const int M = n_tokens, D = c.head_dim, H = c.hidden;
   if (m->lay) {
-    // the session's cache is one page of max_len positions of one sequence
-    std::vector<int32_t> rs((size_t)M, 0), rp((size_t)M), want;
-    std::vector<void *> pools;
-    for (auto &L : m->lay->layers)
-      pools.push_back(L.cache);
-    for (int i = 0; i < M; ++i)
-      rp[(size_t)i] = pos0 + i;
+    std::vector<int32_t> want;
     for (int i = all_rows && logits_host ? 0 : M - 1; i < M; ++i)
       want.push_back(i);
     std::vector<int32_t> nxt(want.size());
+    if (int rc = layered_state_enter(m, pos0)) return rc;
     B200_CUDA(cudaEventRecord(m->ev0, m->stream));
-    if (int rc = layered_rows(m, M, tokens, rs.data(), rp.data(), m->lay->zero, 1, c.max_len, pools.data(), c.max_len,
-                              (int)want.size(), want.data(), logits_host, nxt.data()))
-      return rc;
+    if (int rc = layered_session_rows(m, M, tokens, pos0, (int)want.size(), want.data(), logits_host, nxt.data())) return rc;
     B200_CUDA(cudaEventRecord(m->ev1, m->stream));
     B200_CUDA(cudaStreamSynchronize(m->stream));
     B200_CUDA(cudaEventElapsedTime(&m->last_ms, m->ev0, m->ev1));
     m->rows_fresh = false;
     if (int rc = layered_status(m)) return rc;
+    layered_state_leave(m, pos0 + M);
     if (next_token)
       *next_token = nxt.back();
     return B200_OK;
@@ -1862,7 +1865,7 @@ static int batch_rows(b200_batch *b, int M, const int32_t *tokens, const int32_t
     cudaStream_t st = m->stream;
     B200_CUDA(cudaMemcpyAsync(b->d_table, b->table.data(), b->table.size() * 4, cudaMemcpyHostToDevice, st));
     B200_CUDA(cudaEventRecord(m->ev0, st));
-    if (int rc = layered_rows(m, M, tokens, row_seq, row_pos, b->d_table, b->table_stride, b->page, b->rows_pool.data(),
+    if (int rc = layered_rows(m, M, tokens, row_seq, row_pos, b->d_table, b->table_stride, b->page, b->caches.data(),
                               b->max_context, n_want, want, logits_host, next_host))
       return rc;
     B200_CUDA(cudaEventRecord(m->ev1, st));
@@ -2003,20 +2006,8 @@ int b200_batch_create(b200_model *m, int max_seqs, int page_size, int n_pages, i
   int rc = B200_OK;
   for (auto &p : b->pool)
     if (rc == B200_OK) rc = dev_alloc((void **)&p, pool_bytes);
-  if (m->lay) {
-    const size_t e = m->lay->dtype == B200_F32 ? 4 : 2;
-    for (auto &L : m->lay->layers) {
-      void *p = nullptr;
-      const size_t bytes = (size_t)n_pages * page_size * L.d.row * e;
-      if (rc == B200_OK && L.own()) {
-        rc = dev_alloc(&p, bytes);
-        // padding elements of a row are read and never written
-        if (rc == B200_OK && cudaMemset(p, 0, bytes) != cudaSuccess)
-          rc = fail(B200_ECUDA, "batch_create: cudaMemset failed");
-      }
-      b->rows_pool.push_back(L.own() ? p : b->rows_pool[(size_t)L.source]);
-    }
-  }
+  if (m->lay && rc == B200_OK)
+    rc = layered_caches_create(m, (int64_t)n_pages * page_size, max_seqs, &b->caches);
   if (rc == B200_OK) rc = dev_alloc((void **)&b->d_table, b->table.size() * 4);
   b->max_context = b->table_stride * page_size;
   b->part_rows = max_seqs;
@@ -2036,8 +2027,7 @@ int b200_batch_create(b200_model *m, int max_seqs, int page_size, int n_pages, i
 void b200_batch_destroy(b200_batch *b) {
   if (!b) return;
   for (auto p : b->pool) cudaFree(p);
-  for (size_t i = 0; i < b->rows_pool.size(); ++i)
-    if (b->m->lay->layers[i].own()) cudaFree(b->rows_pool[i]);
+  if (b->m->lay) layered_caches_free(b->m, &b->caches);
   cudaFree(b->d_table); cudaFree(b->d_seq); cudaFree(b->d_pos); cudaFree(b->d_next);
   cudaFree(b->d_part);
   delete b;

@@ -58,33 +58,68 @@ struct Layer {
 // ---- models of described layers ---------------------------------------------------------------
 struct LayeredLayer {
   b200_layer_config cfg{};
-  LatentDims d{};
-  int source = 0;              // the layer whose cache this one attends to (itself, or kv_from)
-  int off_down = 0, off_router = 0;
+  LatentDims d{};              // latent attention
+  HeadsDims h{};               // attention over per-head keys
+  MemoryDims mem{};            // matrix memory
+  int off_down = 0, off_router = 0;                 // parts of `in` (queries first)
+  int off_k = 0, off_v = 0, off_g = -1;
+  int off_mq = 0, off_mk = 0, off_mv = 0, off_mg = 0, off_mi = 0, off_mf = 0;
   int plain = 0;               // rows of `in` before the (gate, up) pairs
   int att = 0;                 // heads * vdim
-  RowMatrix in;                // [q | latent and key part | router | padding | (gate_j, up_j) pairs]
-  RowMatrix out;               // [W_o | W_down] side by side: one contraction over [attention | feed-forward]
+  int mem_col = 0;             // the memory's first column of `out`
+  RowMatrix in;                // every matrix that reads the mixer's input: [q | latent and key part | router | padding |
+                               // (gate_j, up_j) pairs], or [q | k | v | gate | memory's q, k, v, gate, i, f]
+  RowMatrix out;               // [W_o | W_down] or [W_o | memory's W_o] side by side: one contraction
   RowMatrix ukv, uk, uv;       // [W_uk; W_uv], and its two parts
   RowMatrix expert_in, expert_out;   // [experts][(gate_j, up_j) pairs], [experts][W_down]
+  RowMatrix up, down;          // plain feed-forward
+  RowMatrix side_gate, side_proj;    // per-token layer input
   float *norm = nullptr, *down_norm = nullptr, *inv_freq = nullptr;
-  void *cache = nullptr;       // the single-sequence session's rows [max_len][d.row]
+  double *freq = nullptr;
+  float *in_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *mem_norm = nullptr;
+  float *norm_b = nullptr, *norm2 = nullptr, *norm2_b = nullptr, *side_norm = nullptr;
   Gate gate{};
-  bool own() const { return cfg.kv_from < 0; }
+  bool latent() const { return cfg.mixer == B200_MIX_LATENT; }
+  bool heads() const { return cfg.mixer == B200_MIX_HEADS || cfg.mixer == B200_MIX_HEADS_MEMORY; }
+  bool memory() const { return cfg.mixer == B200_MIX_MEMORY || cfg.mixer == B200_MIX_HEADS_MEMORY; }
+  bool own() const { return !latent() || cfg.kv_from < 0; }
+  int64_t row() const { return latent() ? d.row : heads() ? h.row : 0; }   // elements per cached position
+  int64_t state() const { return memory() ? mem.state : 0; }               // f32 values per slot
+};
+struct LayerCache {            // cached rows by position (or page), recurrent state by slot
+  void *rows = nullptr;
+  float *state = nullptr;
+};
+struct LayeredRun {            // one execution of a layer in a step; a looped layer has several
+  int layer = 0;
+  int source = 0;              // the run whose cache this one attends to (itself, or the kv_from layer's)
+  bool again = false;          // the embedding output is added before it
+  LayerCache cache;            // the single-sequence session's: [max_len][row], one slot
 };
 struct LayeredTensor {         // where a named tensor goes
   int rows, cols, dtype;
   void *dst;
   int64_t ld, row0, step, col0;
-  bool set;
+  bool set;                    // or optional
+};
+struct StepPlan {              // the rows of a step by sequence (device arrays)
+  const int4 *segs = nullptr;  // (first row, rows, sequence, first position): n_long of at least kExpandRows rows, then n_short
+  int n_long = 0, n_short = 0;
+  const int4 *tiles = nullptr; // the long segments in tiles of kHeadsQueryTile
+  int n_tiles = 0;
+  const int32_t *singles = nullptr;   // rows outside long segments
+  int n_singles = 0;
+  int ctx = 0;                 // positions that some row may see
 };
 struct LayeredWs {             // activations of up to `rows` rows
   int rows = 0, ctx = 0;
   std::vector<void *> owned;
   float *proj = nullptr, *qabs = nullptr, *part = nullptr, *cat = nullptr, *mid = nullptr, *weight = nullptr;
   int32_t *ids = nullptr;
-  int32_t *row_seq = nullptr, *row_pos = nullptr, *tokens = nullptr;
+  int32_t *row_seq = nullptr, *row_pos = nullptr, *tokens = nullptr, *plan = nullptr;
   float *x = nullptr;
+  float *x2 = nullptr, *y = nullptr, *h32 = nullptr, *mem_o = nullptr;   // sandwich blocks
+  void *q = nullptr;           // rotated queries in the compute type
   // tensor-core path
   bf16 *h16 = nullptr, *cat16 = nullptr, *q16 = nullptr, *x16 = nullptr, *mid16 = nullptr;
   float *expert_y = nullptr;
@@ -92,15 +127,20 @@ struct LayeredWs {             // activations of up to `rows` rows
 };
 struct LayeredState {
   int dtype = B200_F32;
+  b200_stack_config stack{1.f, 0, 0, 1, 0};
   std::vector<LayeredLayer> layers;
+  std::vector<LayeredRun> runs;
   RowMatrix embed;             // also the output head
+  RowMatrix side_embed;        // [vocab][layers * side_dim]
   float *final_norm = nullptr;
   std::map<std::string, LayeredTensor> tensors;
   std::vector<void *> owned;
   int32_t *zero = nullptr;     // sequence 0, page 0: the session's block table
   int ldp = 0, ldc = 0, ldq = 0, max_mid = 0, max_ff = 0, max_top = 0, max_experts = 0;
-  int max_q = 0, max_row = 0, max_kv = 0;
+  int max_q = 0, max_row = 0, max_kv = 0, max_plain = 0, max_mem = 0;
+  bool sandwich = false, memory = false;   // some layer is one / has one
   int window = 0;              // the widest window of all layers, 0: some layer sees everything
+  int state_pos = 0;           // the position the session's recurrent state has reached, -1: unknown
   LayeredWs one, many;         // the captured decode step's rows, and everything else's
   float *x_want = nullptr;     // rows whose logits are asked for
   bf16 *h_want = nullptr;
@@ -182,7 +222,7 @@ struct b200_batch {
   b200_model *m = nullptr;
   int max_seqs = 0, page = 0, n_pages = 0, table_stride = 0;
   std::vector<float *> pool;            // [2 * layers] page pools [n_pages][kv_heads][page][D]
-  std::vector<void *> rows_pool;        // described layers: [layers] page pools [n_pages][page][row] (null: shared)
+  std::vector<b200::LayerCache> caches;   // described layers, per run: page pools [n_pages][page][row], states [max_seqs]
   std::vector<int> first;               // per sequence: first page still held (pages behind every window go back)
   std::vector<int> free_pages;
   std::vector<int> len;                 // per sequence: -1 = unused slot
@@ -201,8 +241,16 @@ void layered_destroy(b200_model *m);
 int layered_ready(b200_model *m);                       // every tensor set?
 int layered_issue_step(b200_model *m, cudaStream_t st); // one decode step of the session from d_state, for capture
 int layered_rows(b200_model *m, int M, const int32_t *tokens, const int32_t *row_seq, const int32_t *row_pos,
-                 const int32_t *table_dev, int table_stride, int page, void *const *pools, int max_ctx, int n_want,
+                 const int32_t *table_dev, int table_stride, int page, const LayerCache *caches, int max_ctx, int n_want,
                  const int32_t *want, float *logits_host, int32_t *next_host);
+int layered_session_rows(b200_model *m, int M, const int32_t *tokens, int pos0, int n_want, const int32_t *want,
+                         float *logits_host, int32_t *next_host);   // on the session's own cache
+// Caches of every run for `positions` cached rows and `slots` recurrent states; and their release.
+int layered_caches_create(const b200_model *m, int64_t positions, int slots, std::vector<LayerCache> *out);
+void layered_caches_free(const b200_model *m, std::vector<LayerCache> *caches);
+// The session is about to run from position pos: its recurrent state must have reached it.
+int layered_state_enter(b200_model *m, int pos);
+void layered_state_leave(b200_model *m, int pos);
 int layered_status(b200_model *m);                      // after a synchronise: did a bounded wait give up?
 int layered_clear_cache(b200_model *m);
 int layered_kv_overflow(b200_model *m, int position, int keep, int *new_position);

@@ -5,7 +5,7 @@
 // Both operands arrive by TMA (cp.async.bulk.tensor, no multicast) as 128-byte-swizzled rows of
 // 64 k; one thread issues tcgen05.mma (128 x 128 or 128 x 256 x 16) into a f32 accumulator in
 // tensor memory; eight warps read it back (tcgen05.ld), apply the epilogue and write whole rows:
-// plain or added to C, f32 or bf16, or the gate of (gate, up) column pairs.  Two CTAs share an
+// plain or added to C, f32 or bf16, with a bias and an activation, or the gate of (gate, up) column pairs.  Two CTAs share an
 // SM, so one's epilogue runs under the other's main loop.  Few output tiles: the k range is split
 // over gridDim.z and a second kernel adds the partial tiles in split order.
 //
@@ -41,6 +41,8 @@ struct Params {
   int64_t ldc;
   int add, pairs;
   Gate gate;
+  const float *bias;
+  RowAct act;
   int stages, splits;
   float *partial;              // [tile][split][128][128]
   const int4 *tiles;           // grouped: (expert, first row, rows, -)
@@ -61,6 +63,14 @@ __device__ __forceinline__ void mma(uint32_t tmem_d, uint64_t da, uint64_t db, u
 
 // Store `cols` staged values of row m from column n on: 1 or 4 at a time.
 __device__ __forceinline__ void store4(const Params &p, int64_t m, int64_t n, float4 v, int valid, bool vec) {
+  if (p.bias != nullptr || p.act.kind != B200_ACT_NONE || p.act.mul != nullptr) {
+    float a[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (e < valid)
+        a[e] = row_act(p.act, p.bias != nullptr ? a[e] + p.bias[n + e] : a[e], m, n + e);
+    v = make_float4(a[0], a[1], a[2], a[3]);
+  }
   if (p.C != nullptr) {
     float *dst = p.C + m * p.ldc + n;
     if (vec && valid == 4) {
@@ -301,6 +311,8 @@ int gemm_bf16_launch(const GemmBf16 &g, void *workspace, cudaStream_t st) {
   p.add = g.add ? 1 : 0;
   p.pairs = g.pairs ? 1 : 0;
   p.gate = g.gate;
+  p.bias = g.bias;
+  p.act = g.act;
   p.splits = 1;
   p.tiles = g.tiles;
   p.n_tiles = g.n_tiles;

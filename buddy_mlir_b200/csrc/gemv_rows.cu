@@ -1,7 +1,10 @@
 // GEMV over plain weight rows (f32 or bfloat16), up to eight activation rows per pass:
 //   y[m, n] (+)= sum_k norm(x)[m, k] * w[n, k]
-// with an optional RMSNorm prologue, a residual sum, and gated (gate, up) row pairs from a given
-// row on, so that one launch serves every projection that reads the same normalised row.
+// with an optional RMSNorm prologue, a bias, an activation, a residual sum, and gated (gate, up) row
+// pairs from a given row on, so that one launch serves every projection that reads the same
+// normalised row.  For one row the prologue also settles the stream: what the sublayer before left
+// (its output still to be normed, the embedding row of a new pass) is added to x by every CTA for
+// itself, and written back by the first.
 // HBM bound: a warp streams R rows with 16-byte loads, each weight byte is read once per pass.
 // And its two forms for a mixture of experts, where the rows to stream are chosen per token on
 // the device (route_row): expert_in_kernel (gate / up of the chosen experts) and
@@ -33,6 +36,10 @@ struct RowsP {
   float *y2;                   // their results
   int64_t ldy2;
   Gate gate;
+  const float *bias;           // per weight row, or null
+  RowAct act;
+  Unsettled late;              // MT == 1, one slab
+  float *x_out;
   int slab;                    // activations staged at a time (a multiple of a block, or all)
 };
 
@@ -70,6 +77,63 @@ __device__ void row_rms(const float *x, int64_t ldx, int K, int rows, float eps,
   __syncthreads();
 }
 
+__device__ __forceinline__ float cta_sum(float s, float *s_red) {
+  s = warp_sum(s);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0)
+    s_red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < kWarps; ++w)
+    t += s_red[w];
+  return t;
+}
+
+// Stage the settled (and normed) row in xs; the first CTA writes the settled row to x_out.
+template <typename T>
+__device__ void stage_settled(const RowsP &p, float4 *xs, float *s_red) {
+  float r = 0.f;
+  if (p.late.y != nullptr) {
+    float s = 0.f;
+    for (int k = threadIdx.x; k < p.K; k += kThreads)
+      s = fmaf(p.late.y[k], p.late.y[k], s);
+    r = 1.0f / sqrtf(cta_sum(s, s_red) / (float)p.K + p.eps);
+  }
+  const T *emb = p.late.embed != nullptr ? reinterpret_cast<const T *>(p.late.embed) + (int64_t)p.late.tokens[0] * p.late.lde : nullptr;
+  const bool keep = blockIdx.x == 0;
+  float s = 0.f;
+  for (int g = threadIdx.x; g < block_pad<T>(p.K) / 4; g += kThreads) {
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int k = 4 * g + e;
+      if (k < p.K) {
+        v[e] = p.x[k];
+        if (p.late.y != nullptr)
+          v[e] = fmaf(p.late.y[k] * r, __ldg(p.late.w + k), v[e]);
+        if (emb != nullptr)
+          v[e] = fmaf(to_float(emb[k]), p.late.scale, v[e]);
+        if (keep)
+          p.x_out[k] = v[e];
+        s = fmaf(v[e], v[e], s);
+      }
+    }
+    xs[stage_slot<T>(g)] = make_float4(v[0], v[1], v[2], v[3]);
+  }
+  if (p.norm_w != nullptr) {
+    const float rx = 1.0f / sqrtf(cta_sum(s, s_red) / (float)p.K + p.eps);
+    for (int g = threadIdx.x; g < block_pad<T>(p.K) / 4; g += kThreads) {   // the groups this thread staged
+      float4 &v = xs[stage_slot<T>(g)];
+      const int k = 4 * g;
+      v.x = k < p.K ? v.x * rx * __ldg(p.norm_w + k) : 0.f;
+      v.y = k + 1 < p.K ? v.y * rx * __ldg(p.norm_w + k + 1) : 0.f;
+      v.z = k + 2 < p.K ? v.z * rx * __ldg(p.norm_w + k + 2) : 0.f;
+      v.w = k + 3 < p.K ? v.w * rx * __ldg(p.norm_w + k + 3) : 0.f;
+    }
+  }
+  __syncthreads();
+}
+
 template <typename T, int MT, int R>
 __global__ void __launch_bounds__(kThreads)
 gemv_rows_kernel(const RowsP p) {
@@ -78,12 +142,15 @@ gemv_rows_kernel(const RowsP p) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int m0 = blockIdx.y * MT, rows = min(MT, p.M - m0);
   const float *x = p.x + (int64_t)m0 * p.ldx;
-  if (p.norm_w != nullptr)
+  const bool settles = MT == 1 && p.x_out != nullptr;
+  if (settles)
+    stage_settled<T>(p, xs, s_red);
+  else if (p.norm_w != nullptr)
     row_rms<MT>(x, p.ldx, p.K, rows, p.eps, s_r, s_red);
   const int Kp = unit_pad<T>(p.K);
   const int xs_ld = p.slab / 4;
   const bool one_slab = p.slab >= Kp;
-  bool staged = false;
+  bool staged = settles;
   const T *w = reinterpret_cast<const T *>(p.w);
   for (int64_t base = (int64_t)blockIdx.x * kWarps * R; base < p.N; base += (int64_t)gridDim.x * kWarps * R) {
     const int64_t row0 = base + warp * R;
@@ -136,7 +203,8 @@ gemv_rows_kernel(const RowsP p) {
           for (int m = 0; m < MT; ++m)
             if (m < rows) {
               float *y = p.y + (int64_t)(m0 + m) * p.ldy + row0 + r;
-              *y = p.add ? *y + acc[r][m] : acc[r][m];
+              const float v = row_act(p.act, p.bias != nullptr ? acc[r][m] + p.bias[row0 + r] : acc[r][m], m0 + m, row0 + r);
+              *y = p.add ? *y + v : v;
             }
     }
   }
@@ -326,28 +394,34 @@ template <typename T> int gemv_rows_pick(RowsP &p, cudaStream_t st) {
 
 } // namespace
 
-int gemv_rows_launch(int dtype, const RowMatrix &w, const float *x, int64_t ldx, int M, const float *norm_w, float eps,
-                     float *y, int64_t ldy, bool add, int pair_from, float *y2, int64_t ldy2, const Gate &gate,
-                     cudaStream_t st) {
+bool gemv_rows_settles(int M, int K) { return M == 1 && block_pad<bf16>(K) <= kSlabBytes / 4; }
+
+int gemv_rows_launch(int dtype, const GemvRows &g, cudaStream_t st) {
   RowsP p{};
-  p.w = w.w;
-  p.ldw = w.ld;
-  p.N = w.N;
-  p.K = w.K;
-  p.M = M;
-  p.x = x;
-  p.ldx = ldx;
-  p.norm_w = norm_w;
-  p.eps = eps;
-  p.y = y;
-  p.ldy = ldy;
-  p.add = add ? 1 : 0;
-  p.pair_from = pair_from;
-  p.y2 = y2;
-  p.ldy2 = ldy2;
-  p.gate = gate;
-  if ((pair_from < w.N) && ((pair_from & 3) || (w.N & 1)))
+  p.w = g.w.w;
+  p.ldw = g.w.ld;
+  p.N = g.w.N;
+  p.K = g.w.K;
+  p.M = g.M;
+  p.x = g.x;
+  p.ldx = g.ldx;
+  p.norm_w = g.norm_w;
+  p.eps = g.eps;
+  p.y = g.y;
+  p.ldy = g.ldy;
+  p.add = g.add ? 1 : 0;
+  p.pair_from = g.pair_from < g.w.N ? g.pair_from : g.w.N;
+  p.y2 = g.y2;
+  p.ldy2 = g.ldy2;
+  p.gate = g.gate;
+  p.bias = g.bias;
+  p.act = g.act;
+  p.late = g.late;
+  p.x_out = g.x_out;
+  if ((p.pair_from < g.w.N) && ((p.pair_from & 3) || (g.w.N & 1)))
     return fail(B200_EINVAL, "gemv_rows: pairs must start at a multiple of four rows");
+  if (g.late.any() != (g.x_out != nullptr) || (g.x_out != nullptr && (!gemv_rows_settles(g.M, p.K) || g.x_out == g.x)))
+    return fail(B200_EINVAL, "gemv_rows: only one row that fits shared memory is settled, into another buffer");
   return dtype == B200_F32 ? gemv_rows_pick<float>(p, st) : gemv_rows_pick<bf16>(p, st);
 }
 

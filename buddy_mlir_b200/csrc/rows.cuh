@@ -143,6 +143,45 @@ __device__ __forceinline__ float gate_pair(const Gate &p, float g, float u) {
   return (g / (1.0f + expf(-p.slope * g))) * (u + p.offset);
 }
 
+// What a contraction's epilogue does to a result (row m, column n) besides the bias: an activation,
+// and a factor mul[row[m]][n] (a table in the compute type).
+struct RowAct {
+  int kind;                    // B200_ACT_*
+  const void *mul;             // null: none
+  int mul_f32;
+  int64_t ld;
+  const int32_t *row;
+};
+__device__ __forceinline__ float activate(int kind, float z) {
+  if (kind == B200_ACT_RELU2) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+  }
+  if (kind == B200_ACT_GELU_TANH)
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z;
+}
+__device__ __forceinline__ float row_act(const RowAct &a, float z, int64_t m, int64_t n) {
+  z = activate(a.kind, z);
+  if (a.mul != nullptr) {
+    const int64_t i = (int64_t)a.row[m] * a.ld + n;
+    z *= a.mul_f32 ? reinterpret_cast<const float *>(a.mul)[i] : __bfloat162float(reinterpret_cast<const bf16 *>(a.mul)[i]);
+  }
+  return z;
+}
+
+// What is still to be added to rows of the residual stream: RMSNorm(y) * w (y null: nothing), and the
+// scaled embedding row of the token (embed null: nothing; a table in the compute type).
+struct Unsettled {
+  const float *y;              // rows as long as the stream's, tight
+  const float *w;
+  const void *embed;
+  int64_t lde;
+  float scale;
+  const int32_t *tokens;
+  __host__ __device__ bool any() const { return y != nullptr || embed != nullptr; }
+};
+
 // mma.sync building blocks
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);

@@ -3,10 +3,10 @@ architecture is known."""
 import json
 import os
 
-from . import config, talazen
+from . import butolorn, config, talazen
 
 # architecture name in config.json -> parser of that file
-ARCHITECTURES = {"Talazen": talazen.parse}
+ARCHITECTURES = {"Butolorn": butolorn.parse, "Talazen": talazen.parse}
 
 # shapes of the blob-loaded models by name
 SHAPES = {c.name: c for c in (config.DEEPSEEK_R1_1P5B, config.QWEN3_8B, config.TINY_QWEN2,

@@ -273,39 +273,83 @@ int b200_model_create(const b200_model_config *cfg, b200_model **out);
 
 /* ---- models given as a list of described layers ----------------------------
  * A decoder whose layers differ: each layer names its token mixer and its
- * feed-forward with their sizes and constants.  A layer is a parallel block,
- * x += mixer(h) + ff(h) with h = RMSNorm(x); the output is RMSNorm and the
- * transposed embedding table.  (No counterpart in buddy-mlir.)  The handle is
- * an ordinary b200_model: decode, generate, prefill and the batch calls take
- * it; tensors are loaded by name (b200_model_set_tensor). */
-enum { B200_MIX_LATENT = 0 };
-enum { B200_FF_NONE = 0, B200_FF_GATED = 1, B200_FF_EXPERTS = 2 };
+ * feed-forward with their sizes and constants.  (No counterpart in buddy-mlir.)
+ * The handle is an ordinary b200_model: decode, generate, prefill and the batch
+ * calls take it; tensors are loaded by name (b200_model_set_tensor).  The output
+ * is RMSNorm and the transposed embedding table. */
+enum {
+  B200_MIX_LATENT = 0,  /* attention over a cached low-rank latent with a rotated
+                         * key part that all heads share                       */
+  B200_MIX_HEADS = 1,   /* attention over keys and values cached per head      */
+  B200_MIX_MEMORY = 2,  /* matrix memory: a gated recurrent [dim][vdim] state
+                         * per head                                            */
+  B200_MIX_HEADS_MEMORY = 3 /* both side by side on the same input, summed     */
+};
+enum {
+  B200_BLOCK_PARALLEL = 0, /* x += mixer(h) + ff(h), h = RMSNorm(x)            */
+  B200_BLOCK_SANDWICH = 1  /* x += norm1b(mixer(norm1(x))), then
+                            * x += norm2b(ff(norm2(x)))                        */
+};
+enum { B200_FF_NONE = 0, B200_FF_GATED = 1, B200_FF_EXPERTS = 2, B200_FF_PLAIN = 3 };
+enum { B200_ACT_NONE = 0, B200_ACT_RELU2 = 1, B200_ACT_GELU_TANH = 2 };
 typedef struct {
-  int32_t mixer;     /* B200_MIX_LATENT: attention over a cached low-rank latent
-                      * with a rotated key part that all heads share           */
-  int32_t heads, dim, rot_dim, vdim; /* per head: unrotated and rotated query /
-                      * key sizes, value size (rotation: interleaved pairs)    */
-  int32_t kv_rank;   /* latent size                                            */
+  int32_t mixer;     /* B200_MIX_*                                             */
+  int32_t heads, dim, rot_dim, vdim; /* per head.  Latent: unrotated and rotated
+                      * query / key sizes, value size.  Heads: query / key size,
+                      * how many of its first dimensions are rotated, value size */
+  int32_t kv_rank;   /* latent: its size                                       */
   int32_t window;    /* sliding window in tokens, 0: everything before         */
-  int32_t kv_from;   /* attend to that earlier layer's cache, -1: own cache    */
+  int32_t kv_from;   /* latent: attend to that earlier layer's cache, -1: own  */
   float scale, rot_base;
   int32_t ff_kind;   /* B200_FF_*                                              */
   int32_t ff;        /* width of the feed-forward, or of one expert            */
   int32_t experts, top;
-  float limit, gate_slope, up_offset; /* g = min(g, limit), u = clamp(u, -limit, limit),
-                      * g * sigmoid(gate_slope * g) * (u + up_offset)          */
+  float limit, gate_slope, up_offset; /* gated: g = min(g, limit), u = clamp(u,
+                      * -limit, limit), g * sigmoid(gate_slope * g) * (u + up_offset) */
+  int32_t block;     /* B200_BLOCK_*; latent layers are parallel blocks, the
+                      * others sandwiches                                      */
+  int32_t ff_act;    /* plain: down(act(up x)), B200_ACT_*                     */
+  /* attention over per-head keys */
+  int32_t kv_heads;
+  int32_t rot_halves; /* rotation pairs (i, i + rot_dim/2), 0: (2i, 2i + 1)    */
+  int32_t qkv_bias;
+  int32_t qk_norm;   /* RMSNorm over the whole query and the whole key projection */
+  int32_t out_gate;  /* heads times sigmoid(W_g h) before the output projection */
+  float sink;        /* score of one more softmax entry without a value, -inf: none */
+  float mix_scale;   /* factor on this mixer's output                          */
+  /* matrix memory; log gates i = cap tanh(z / cap), f = logsigmoid(cap tanh(z / cap)),
+   * o = S^T q / (max(|n q|, exp(-m)) + mem_floor), normed per head, gated     */
+  int32_t mem_heads, mem_dim, mem_vdim;
+  float mem_cap, mem_q_scale, mem_floor, mem_mix_scale;
 } b200_layer_config;
-/* cfg: hidden, n_layers, vocab, max_len and eps are read.  dtype: B200_BF16
- * (weights, cache and matrix operands in bfloat16; norms, router, softmax,
- * residual and all sums in f32) or B200_F32 (everything in f32). */
+/* What concerns the stack of layers. */
+typedef struct {
+  float embed_scale; /* factor on the embedding rows                           */
+  int32_t loop_start, loop_stop, loop_times; /* layers start .. stop-1 run `times`
+                      * times with caches of their own per pass; the embedding
+                      * output is added before every pass but the first        */
+  int32_t side_dim;  /* per-token layer input: x += RMSNorm(proj(gelu(gate x) * e)),
+                      * e = the layer's part of a row of "side.embed"; 0: none */
+} b200_stack_config;
+/* cfg: hidden, n_layers, vocab, max_len and eps are read.  stack: null for
+ * scale 1, no loop, no per-token input.  dtype: B200_BF16 (weights, cache and
+ * matrix operands in bfloat16; norms, router, softmax, recurrent state, residual
+ * and all sums in f32) or B200_F32 (everything in f32). */
 int b200_model_create_layered(const b200_model_config *cfg,
+                              const b200_stack_config *stack,
                               const b200_layer_config *layers, int dtype,
                               b200_model **out);
 /* A named tensor from HOST memory, row-major [rows, cols] = [out, in] (vectors:
  * rows = 1), dtype B200_BF16 or B200_F32.  Names: "embed", "final.norm", and
  * per layer i "l<i>.norm1", "l<i>.mix.{q,dkv,dkv.norm,uk,uv,o}",
  * "l<i>.mlp.{gate,up,down}" or "l<i>.mlp.router" and
- * "l<i>.mlp.e<j>.{gate,up,down}". */
+ * "l<i>.mlp.e<j>.{gate,up,down}".  Heads: "l<i>.mix.{q,k,v,o}" with "q.b",
+ * "k.b", "v.b", "q.norm", "k.norm", "g" where configured; memory:
+ * "l<i>.mix.{q,k,v,g,o,norm,i,i.b,f,f.b}"; side by side, "mix.left." and
+ * "mix.right." in their place.  Sandwich: "l<i>.{norm1,norm1b,norm2,norm2b}"
+ * (the last two may be left out of a layer without a feed-forward); plain
+ * feed-forward "l<i>.mlp.{up,down}"; per-token input "side.embed" and
+ * "l<i>.side.{gate,proj,norm}". */
 int b200_model_set_tensor(b200_model *m, const char *name, int dtype,
                           const void *host, int64_t rows, int64_t cols);
 /* Residual stream of the rows of the last prefill / batch call of such a model
