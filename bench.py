@@ -558,6 +558,35 @@ def layered_model(name, window=None):
     return s
 
 
+def butolorn_model(name):
+    """A Butolorn of the same width, depth and heads: layers of attention and of sink attention (half
+    the heads) beside a matrix memory (the other half's width) in turn, a two-matrix feed-forward as
+    large as the other models' three, a per-token input of 64."""
+    from buddy_mlir_b200 import butolorn
+    from buddy_mlir_b200.session import ModelSession
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    import plain_butolorn
+    H, heads, kvh, ff, _, _, _ = LAYERED_SHAPES[name]
+    L = LAYERED
+
+    def att(n, kv, rot):
+        return {"heads": n, "kv_heads": kv, "dim": L["dim"], "vdim": L["vdim"], "rot": {"base": 10000.0, "dims": rot},
+                "scale": L["dim"] ** -0.5}
+    mlp = {"kind": "dense", "ff": ff * 3 // 2}
+    both = {"left": att(heads // 2, max(1, kvh // 2), 64), "left_scale": 1.0, "right_scale": 1.0,
+            "right": {"heads": heads // 4, "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+    layers = [{"type": "parallel", "mixer": both, "mlp": mlp} if i % 2 == 0 else
+              {"type": "attention", "mixer": att(heads, kvh, 128), "mlp": mlp} for i in range(L["layers"])]
+    cfg = {"architecture": "Butolorn", "width": H, "vocab": L["vocab"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+           "layers": layers, "token_side": {"dim": 64}}
+    pool = np.random.default_rng(SEED_W).standard_normal(1 << 22).astype(np.float32) * 0.02
+    big = np.tile((pool.view(np.uint32) >> 16).astype(np.uint16), 64)
+    s = ModelSession(butolorn.parse(cfg, "bfloat16", 4096))
+    s.load_named({k: (np.ones(shape, np.float32) if len(shape) == 1 else big[:shape[0] * shape[1]].reshape(shape))
+                  for k, shape in plain_butolorn.tensor_shapes(cfg).items()})
+    return s
+
+
 def uniform_model(name):
     """The int8 uniform-attention model of the same width, depth, heads and active feed-forward."""
     from buddy_mlir_b200 import _lib
@@ -621,7 +650,7 @@ def session_numbers(s, steps=64):
 
 
 def run_layered_only(args):
-    """--layered: prefill and decode of models of described layers (Talazen, bfloat16) at the sizes of
+    """--layered: prefill and decode of models of described layers (Talazen, Butolorn, bfloat16) at the sizes of
     LAYERED_SHAPES, beside the uniform int8 model of equal size (one JSON line)."""
     import torch
     from buddy_mlir_b200 import _lib
@@ -634,7 +663,7 @@ def run_layered_only(args):
     sampler.start()
     for name in ([args.layered_shape] if args.layered_shape else LAYERED_SHAPES):
         out[name] = {}
-        for kind, make in (("talazen_bf16", layered_model), ("uniform_int8", uniform_model)):
+        for kind, make in (("butolorn_bf16", butolorn_model), ("talazen_bf16", layered_model), ("uniform_int8", uniform_model)):
             if args.layered_kind and args.layered_kind != kind:
                 continue
             s = make(name)
@@ -779,9 +808,9 @@ def main():
     ap.add_argument("--batch-only", action="store_true", help="batched decode (64 sequences, paged KV) + a 2048-token prefill")
     ap.add_argument("--w8a8-only", action="store_true", help="the w8a8 arithmetic on the 1.5B int8 model: prefill and decode")
     ap.add_argument("--layered", action="store_true",
-                    help="models of described layers (Talazen) beside the uniform model of equal size: prefill, decode, batched decode")
+                    help="models of described layers (Talazen, Butolorn) beside the uniform model of equal size: prefill, decode, batched decode")
     ap.add_argument("--layered-shape", default=None, help="with --layered: one of LAYERED_SHAPES")
-    ap.add_argument("--layered-kind", default=None, help="with --layered: talazen_bf16 or uniform_int8 alone")
+    ap.add_argument("--layered-kind", default=None, help="with --layered: butolorn_bf16, talazen_bf16 or uniform_int8 alone")
     ap.add_argument("--gemm-shape", default=None, help="with --gemm-only: one shape of GEMM_SHAPES")
     ap.add_argument("--resident-only", action="store_true",
                     help="skip the isolated-GEMV, end-to-end and CPU legs (for profiler captures)")

@@ -263,7 +263,7 @@ MemoryDims memory_dims(const b200_layer_config &c) {
   d.heads = c.mem_heads; d.dim = c.mem_dim; d.vdim = c.mem_vdim;
   d.cap = c.mem_cap; d.q_scale = c.mem_q_scale; d.floor = c.mem_floor;
   d.tiles = (d.vdim + 31) / 32;
-  d.head_state = pad_to((int64_t)d.dim * d.tiles * 32 + (int64_t)d.tiles * (d.dim + 1), 32);
+  d.head_state = pad_to((int64_t)d.dim * d.tiles * 32 + (int64_t)d.tiles * (d.dim + 2), 32);
   d.state = d.heads * d.head_state;
   return d;
 }

@@ -13,7 +13,8 @@
 //                        terms and are summed in f32; F and a are kept in double.
 //
 // State of a slot, per head: S [dim][tiles * 32], then for each 32-column tile its own copy of
-// n [dim], then of m, so that the CTAs of a head need nothing from one another.
+// n [dim], then of m, so that the CTAs of a head need nothing from one another.  m is a sum of as
+// many terms as there are tokens and is taken exponentials of: it is kept as two f32 (a double).
 #include "layered.cuh"
 #include "rows.cuh"
 
@@ -25,6 +26,12 @@ namespace {
 
 __device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+__device__ __forceinline__ double load_max(const float *p) { return (double)p[0] + (double)p[1]; }
+__device__ __forceinline__ void store_max(float *p, double m) {
+  p[0] = (float)m;
+  p[1] = (float)(m - (double)p[0]);
+}
 
 // grid (segments * heads, tiles), 8 warps: a lane per column, a warp's rows d = warp + 8 r
 template <int R>
@@ -38,7 +45,7 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
   const int4 seg = segs[blockIdx.x / d.heads];     // first row, rows, slot
   float *st = states + (int64_t)seg.z * d.state + (int64_t)h * d.head_state;
   float *sS = st + col, *sN = st + (int64_t)d.dim * d.tiles * 32 + (int64_t)tile * d.dim;
-  float *sM = st + (int64_t)d.dim * d.tiles * 32 + (int64_t)d.tiles * d.dim + tile;
+  float *sM = st + (int64_t)d.dim * d.tiles * 32 + (int64_t)d.tiles * d.dim + 2 * tile;
   const int64_t ld = d.tiles * 32;
   const bool fresh = row_pos[seg.x] == 0;
   float S[R], n[(DM + 255) / 256];
@@ -48,7 +55,7 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
 #pragma unroll
   for (int i = 0; i < (DM + 255) / 256; ++i)
     n[i] = !fresh && tid + 256 * i < d.dim ? sN[tid + 256 * i] : 0.f;
-  float m = fresh ? 0.f : *sM;
+  double m = fresh ? 0.0 : load_max(sM);
   for (int t = 0; t < seg.y; ++t) {
     const int b = t & 1;
     const float *p = in.proj + (int64_t)(seg.x + t) * in.ldp;
@@ -58,7 +65,8 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
     }
     const float v = col < d.vdim ? p[in.off_v + h * d.vdim + col] : 0.f;
     const float ig = capped(p[in.off_i + h], d.cap), fg = log_sigmoid(capped(p[in.off_f + h], d.cap));
-    const float nm = fmaxf(fg + m, ig), keep = expf(fg + m - nm), add = expf(ig - nm);
+    const double fm = (double)fg + m, nm = fmax(fm, (double)ig);
+    const float keep = expf((float)(fm - nm)), add = expf((float)((double)ig - nm));
     m = nm;
     __syncthreads();
     float acc = 0.f;
@@ -86,7 +94,7 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
         a += s_o[b][w][lane];
         c += s_n[b][w];
       }
-      o[(int64_t)(seg.x + t) * ldo + h * d.vdim + col] = a / (fmaxf(fabsf(c), expf(-m)) + d.floor);
+      o[(int64_t)(seg.x + t) * ldo + h * d.vdim + col] = a / (fmaxf(fabsf(c), expf((float)-m)) + d.floor);
     }
   }
 #pragma unroll
@@ -98,7 +106,7 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
     if (tid + 256 * i < d.dim)
       sN[tid + 256 * i] = n[i];
   if (tid == 0)
-    *sM = m;
+    store_max(sM, m);
 }
 
 constexpr int kChunk = 64;
@@ -147,7 +155,7 @@ memory_chunk_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, con
     }
   });
   if (tid == 0)
-    s_m = fresh ? 0.0 : (double)sM[tile0];
+    s_m = fresh ? 0.0 : load_max(sM + 2 * tile0);
   for (int i = tid; i < (2 * L * LK + 3 * L * LV + 2 * DK * LV) / 8; i += 128)
     reinterpret_cast<uint4 *>(smc)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
@@ -384,7 +392,7 @@ memory_chunk_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, con
     }
   });
   if (tid >= tile0 && tid < tile1)
-    sM[tid] = (float)s_m;
+    store_max(sM + 2 * tid, s_m);
 }
 
 template <int R>
