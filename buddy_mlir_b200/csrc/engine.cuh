@@ -107,6 +107,9 @@ struct StepPlan {              // the rows of a step by sequence (device arrays)
   int n_long = 0, n_short = 0;
   const int4 *tiles = nullptr; // the long segments in tiles of kHeadsQueryTile
   int n_tiles = 0;
+  const int4 *chunks = nullptr;       // and in chunks of kMemoryChunk, of which segment i has those from chunk0[i] on
+  const int32_t *chunk0 = nullptr;
+  int n_chunks = 0;
   const int32_t *singles = nullptr;   // rows outside long segments
   int n_singles = 0;
   int ctx = 0;                 // positions that some row may see
@@ -137,7 +140,8 @@ struct LayeredState {
   std::vector<void *> owned;
   int32_t *zero = nullptr;     // sequence 0, page 0: the session's block table
   int ldp = 0, ldc = 0, ldq = 0, max_mid = 0, max_ff = 0, max_top = 0, max_experts = 0;
-  int max_q = 0, max_row = 0, max_kv = 0, max_plain = 0, max_mem = 0;
+  int max_q = 0, max_row = 0, max_kv = 0, max_plain = 0, max_mem = 0, max_mem_heads = 0;
+  int64_t max_state = 0;
   bool sandwich = false, memory = false;   // some layer is one / has one
   int window = 0;              // the widest window of all layers, 0: some layer sees everything
   int state_pos = 0;           // the position the session's recurrent state has reached, -1: unknown
@@ -150,6 +154,9 @@ struct LayeredState {
   void *gemm_ws = nullptr;     // error word, split-k partial tiles
   bf16 *keys16 = nullptr, *kv16 = nullptr;   // a prompt segment's cache rows, and their expanded keys and values
   int64_t key_rows = 0;
+  float *mem_U = nullptr;      // the matrix memory's states between the chunks of a step
+  double *mem_meta = nullptr;
+  int64_t mem_chunks = 0;
 };
 struct RowSegment {            // consecutive rows of one sequence
   int row0, n, seq, pos0;

@@ -142,6 +142,14 @@ gemv_rows_kernel(const RowsP p) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int m0 = blockIdx.y * MT, rows = min(MT, p.M - m0);
   const float *x = p.x + (int64_t)m0 * p.ldx;
+  {
+    // the CTA's first weight rows start on their way to L2 under the prologue
+    const int64_t row = (int64_t)blockIdx.x * kWarps * R + warp * R + lane;
+    if (lane < R && row < p.N) {
+      const T *w = reinterpret_cast<const T *>(p.w) + row * p.ldw;
+      asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(w), "r"((uint32_t)(unit_pad<T>(p.K) * sizeof(T))) : "memory");
+    }
+  }
   const bool settles = MT == 1 && p.x_out != nullptr;
   if (settles)
     stage_settled<T>(p, xs, s_red);

@@ -29,7 +29,7 @@ __device__ __forceinline__ void turn_table(float *cs, const double *freq, int ha
   constexpr double kTurn = 6.283185307179586476925286766559;
   for (int i = t; i < half; i += nt) {
     const double a = (double)pos * freq[i];
-    sincosf((float)(a - rint(a / kTurn) * kTurn), &cs[half + i], &cs[i]);
+    sincosf((float)(a - rint(a * (1.0 / kTurn)) * kTurn), &cs[half + i], &cs[i]);
   }
 }
 
@@ -46,27 +46,29 @@ __device__ __forceinline__ float turned(const HeadsDims &d, const float *x, int 
   return (c & 1) ? at(c) * cs[i] + at(c - 1) * cs[half + i] : at(c) * cs[i] - at(c + 1) * cs[half + i];
 }
 
-// grid M, a CTA per row
+// grid (M, y): a row's query, key and value heads are dealt to the warps of its y CTAs
 template <typename T>
 __global__ void __launch_bounds__(256)
 heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const CacheView cv) {
   extern __shared__ float s_cs[];
   __shared__ float s_red[16];
-  const int m = blockIdx.x, tid = threadIdx.x;
+  const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
   const float *src = in.proj + (int64_t)m * in.ldp, *ks = src + in.off_k, *vs = src + in.off_v;
   const int pos = cv.row_pos[m];
   turn_table(s_cs, in.freq, d.rot >> 1, pos, tid, 256);
   float rq = 1.f, rk = 1.f;
-  const int nq = d.heads * d.dim, nk = d.kv * d.dim;
   if (in.q_norm != nullptr) {
+    const int nq = d.heads * d.dim, nk = d.kv * d.dim;
     float a = 0.f, b = 0.f;
+#pragma unroll 4
     for (int i = tid; i < nq; i += 256)
       a = fmaf(src[i], src[i], a);
+#pragma unroll 4
     for (int i = tid; i < nk; i += 256)
       b = fmaf(ks[i], ks[i], b);
     a = warp_sum(a);
     b = warp_sum(b);
-    if ((tid & 31) == 0) {
+    if (lane == 0) {
       s_red[tid >> 5] = a;
       s_red[8 + (tid >> 5)] = b;
     }
@@ -80,22 +82,24 @@ heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const Cach
     rk = 1.0f / sqrtf(b / (float)nk + in.eps);
   }
   __syncthreads();
-  T *qd = q + (int64_t)m * d.heads * d.dimp;
-  for (int i = tid; i < d.heads * d.dimp; i += 256) {
-    const int h = i / d.dimp, c = i - h * d.dimp;
-    qd[i] = from_float<T>(c < d.dim ? turned(d, src + h * d.dim, c, rq, in.q_norm ? in.q_norm + h * d.dim : nullptr, s_cs) : 0.f);
-  }
   T *row = pool + cache_row(cv, cv.row_seq[m], pos) * d.row;
-  for (int i = tid; i < d.kv * d.dimp; i += 256) {
-    const int h = i / d.dimp, c = i - h * d.dimp;
-    if (c < d.dim)
-      row[i] = from_float<T>(turned(d, ks + h * d.dim, c, rk, in.k_norm ? in.k_norm + h * d.dim : nullptr, s_cs));
-  }
-  row += d.kv * d.dimp;
-  for (int i = tid; i < d.kv * d.vdimp; i += 256) {
-    const int h = i / d.vdimp, c = i - h * d.vdimp;
-    if (c < d.vdim)
-      row[i] = from_float<T>(vs[h * d.vdim + c]);
+  for (int u = blockIdx.y * 8 + (tid >> 5); u < d.heads + 2 * d.kv; u += gridDim.y * 8) {
+    if (u < d.heads) {
+      T *dst = q + ((int64_t)m * d.heads + u) * d.dimp;
+#pragma unroll 4
+      for (int c = lane; c < d.dimp; c += 32)
+        dst[c] = from_float<T>(c < d.dim ? turned(d, src + u * d.dim, c, rq, in.q_norm ? in.q_norm + u * d.dim : nullptr, s_cs) : 0.f);
+    } else if (u < d.heads + d.kv) {
+      const int h = u - d.heads;
+#pragma unroll 4
+      for (int c = lane; c < d.dim; c += 32)
+        row[h * d.dimp + c] = from_float<T>(turned(d, ks + h * d.dim, c, rk, in.k_norm ? in.k_norm + h * d.dim : nullptr, s_cs));
+    } else {
+      const int h = u - d.heads - d.kv;
+#pragma unroll 4
+      for (int c = lane; c < d.vdim; c += 32)
+        row[d.kv * d.dimp + h * d.vdimp + c] = from_float<T>(vs[h * d.vdim + c]);
+    }
   }
 }
 
@@ -385,50 +389,84 @@ struct CatRow {
 };
 __device__ __forceinline__ float gated(float v, const float *g) { return g != nullptr ? v / (1.0f + expf(-*g)) : v; }
 
-// grid (rows, attention heads + memory heads), 128 threads
+// grid (rows, attention heads + memory heads / 4), 128 threads: four warps share the splits of an
+// attention head, or take a memory head each
 __global__ void __launch_bounds__(128)
 mix_finish_kernel(const MixFinish f) {
-  __shared__ float s_w[kMaxSplits], s_red[4];
-  const int m = f.rows ? f.rows[blockIdx.x] : (int)blockIdx.x, tid = threadIdx.x;
+  __shared__ float s_w[kMaxSplits];
+  __shared__ float4 s_o[4][32];
+  const int m = f.rows ? f.rows[blockIdx.x] : (int)blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const CatRow out{f.cat ? f.cat + (int64_t)m * f.ldc : nullptr, f.cat16 ? f.cat16 + (int64_t)m * f.ldc : nullptr};
   const float *proj = f.proj + (int64_t)m * f.ldp;
   int h = blockIdx.y;
   if (h < f.n_heads) {
     const HeadsDims &d = f.h;
-    const float *part = f.part + ((int64_t)blockIdx.x * d.heads + h) * f.splits * (d.vdimp + 4);
-    const float *ml = part + d.vdimp;
+    const int64_t ld = d.vdimp + 4;
+    const float *part = f.part + ((int64_t)blockIdx.x * d.heads + h) * f.splits * ld;
+    // maxima and sums, two splits per lane (kMaxSplits = 64), the same in every warp
     const float sink = d.sink * kLog2e;
-    float mx = sink;
-    for (int s = 0; s < f.splits; ++s)
-      mx = fmaxf(mx, ml[s * (d.vdimp + 4)]);
-    for (int s = tid; s < f.splits; s += 128)
-      s_w[s] = ml[s * (d.vdimp + 4) + 1] > 0.f ? exp2f(ml[s * (d.vdimp + 4)] - mx) : 0.f;
-    __syncthreads();
-    float l = exp2f(sink - mx);
-    for (int s = 0; s < f.splits; ++s)
-      l = fmaf(s_w[s], ml[s * (d.vdimp + 4) + 1], l);
+    float ms[2], ls[2], mx = sink;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int sp = lane + 32 * i;
+      ms[i] = sp < f.splits ? part[sp * ld + d.vdimp] : -INFINITY;
+      ls[i] = sp < f.splits ? part[sp * ld + d.vdimp + 1] : 0.f;
+      mx = fmaxf(mx, ms[i]);
+    }
+    mx = warp_max(mx);
+    float l = 0.f;
+    int live = 0;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float w = ls[i] > 0.f ? exp2f(ms[i] - mx) : 0.f;
+      if (warp == 0)
+        s_w[lane + 32 * i] = w;
+      l = fmaf(w, ls[i], l);
+      const unsigned some = __ballot_sync(0xffffffffu, ls[i] > 0.f);
+      if (some)
+        live = 32 * i + 32 - __clz(some);
+    }
+    l = warp_sum(l) + exp2f(sink - mx);
     const float inv = f.h_scale / l;
-    for (int c = tid; c < d.vdim; c += 128) {
-      float a = 0.f;
-      for (int s = 0; s < f.splits; ++s)
-        if (s_w[s] > 0.f)
-          a = fmaf(s_w[s], part[s * (d.vdimp + 4) + c], a);
-      out.set(h * d.vdim + c, gated(a * inv, f.off_g >= 0 ? proj + f.off_g + h * d.vdim + c : nullptr));
+    __syncthreads();
+    for (int c0 = 0; c0 < d.vdimp; c0 += 128) {
+      const int c = c0 + lane * 4;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < d.vdimp)
+#pragma unroll 4
+        for (int sp = warp; sp < live; sp += 4) {
+          const float w = s_w[sp];
+          if (w > 0.f) {       // an empty split has no values
+            const float4 v = *reinterpret_cast<const float4 *>(part + sp * ld + c);
+            a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+          }
+        }
+      s_o[warp][lane] = a;
+      __syncthreads();
+      const int cc = c0 + tid;
+      if (cc < d.vdim) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w)
+          v += reinterpret_cast<const float *>(s_o[w])[tid];
+        out.set(h * d.vdim + cc, gated(v * inv, f.off_g >= 0 ? proj + f.off_g + h * d.vdim + cc : nullptr));
+      }
+      __syncthreads();
     }
     return;
   }
-  h -= f.n_heads;
+  h = (h - f.n_heads) * 4 + warp;
+  if (h >= f.n_mem)
+    return;
   const int vd = f.mem_vdim;
   const float *o = f.mem_o + (int64_t)m * f.ldo + h * vd;
   float s = 0.f;
-  for (int c = tid; c < vd; c += 128)
+#pragma unroll 4
+  for (int c = lane; c < vd; c += 32)
     s = fmaf(o[c], o[c], s);
-  s = warp_sum(s);
-  if ((tid & 31) == 0)
-    s_red[tid >> 5] = s;
-  __syncthreads();
-  const float r = f.m_scale / sqrtf((s_red[0] + s_red[1] + s_red[2] + s_red[3]) / (float)vd + f.eps);
-  for (int c = tid; c < vd; c += 128)
+  const float r = f.m_scale / sqrtf(warp_sum(s) / (float)vd + f.eps);
+#pragma unroll 4
+  for (int c = lane; c < vd; c += 32)
     out.set(f.mem_col + h * vd + c, gated(o[c] * r * f.mem_norm[h * vd + c], proj + f.off_mg + h * vd + c));
 }
 
@@ -694,10 +732,12 @@ int64_t heads_scratch_floats(const HeadsDims &d, int rows, int splits) {
 int heads_prep_launch(int dtype, const HeadsDims &d, const HeadsIn &in, int M, void *q, void *pool, const CacheView &cv,
                       cudaStream_t st) {
   const size_t smem = (size_t)d.rot * 4 + 16;
+  const int units = (d.heads + 2 * d.kv + 7) / 8;
+  const dim3 grid(M, std::max(1, std::min(units, 592 / M)));
   if (dtype == B200_F32)
-    heads_prep_kernel<float><<<M, 256, smem, st>>>(d, in, (float *)q, (float *)pool, cv);
+    heads_prep_kernel<float><<<grid, 256, smem, st>>>(d, in, (float *)q, (float *)pool, cv);
   else
-    heads_prep_kernel<bf16><<<M, 256, smem, st>>>(d, in, (bf16 *)q, (bf16 *)pool, cv);
+    heads_prep_kernel<bf16><<<grid, 256, smem, st>>>(d, in, (bf16 *)q, (bf16 *)pool, cv);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -728,7 +768,7 @@ int heads_attend_launch(int dtype, const HeadsDims &d, const void *q, const int3
 }
 
 int mix_finish_launch(const MixFinish &f, int M, cudaStream_t st) {
-  mix_finish_kernel<<<dim3(M, f.n_heads + f.n_mem), 128, 0, st>>>(f);
+  mix_finish_kernel<<<dim3(M, f.n_heads + (f.n_mem + 3) / 4), 128, 0, st>>>(f);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

@@ -418,6 +418,8 @@ int build_sandwich(LayeredState *s, LayeredLayer &L, int i, int W) {
   s->max_q = std::max(s->max_q, d.heads * d.dimp);
   s->max_row = std::max(s->max_row, (int)L.row());
   s->max_mem = std::max(s->max_mem, (int)pad_to(mv, 4));
+  s->max_mem_heads = std::max(s->max_mem_heads, e.heads);
+  s->max_state = std::max(s->max_state, e.state);
   return B200_OK;
 }
 
@@ -488,7 +490,7 @@ int build_layer(LayeredState *s, LayeredLayer &L, int i, int W) {
 // From this many rows on a bfloat16 model contracts on the tensor cores; a run of consecutive
 // rows of one sequence of this length expands its keys (latent_prefill.cu).
 constexpr int kDenseRows = 9, kExpandRows = 17;
-constexpr int kPlanInts = 10;            // of a StepPlan, per row: segments, tiles, single rows
+constexpr int kPlanInts = 10;            // of a StepPlan, per row: segments, tiles, chunks, single rows
 
 bool dense(const LayeredState *s, int M) { return s->dtype == B200_BF16 && M >= kDenseRows; }
 
@@ -753,6 +755,23 @@ int reserve_keys(b200_model *m, int64_t n) {
   return B200_OK;
 }
 
+// Room for the matrix memory's states between n chunks.
+int reserve_chunks(b200_model *m, int64_t n) {
+  LayeredState *s = m->lay;
+  if (n <= s->mem_chunks)
+    return B200_OK;
+  B200_CUDA(cudaStreamSynchronize(m->stream));
+  cudaFree(s->mem_U);
+  cudaFree(s->mem_meta);
+  s->mem_U = nullptr;
+  s->mem_meta = nullptr;
+  s->mem_chunks = 0;
+  if (int rc = dev_alloc((void **)&s->mem_U, (size_t)n * s->max_state * 4)) return rc;
+  if (int rc = dev_alloc((void **)&s->mem_meta, (size_t)n * s->max_mem_heads * 3 * 8)) return rc;
+  s->mem_chunks = n;
+  return B200_OK;
+}
+
 // The attention of one layer for all rows, bf16: long runs of a sequence over expanded keys,
 // what lies between them in the single-query form.
 int dense_attention(b200_model *m, LayeredWs &ws, LayeredLayer &L, int M, const CacheView &cv,
@@ -836,8 +855,11 @@ int dense_sandwich(b200_model *m, LayeredWs &ws, Stream &z, const LayeredLayer &
   if (L.memory()) {
     const MemoryIn in = memory_in(s, ws, L);
     const int chunked = memory_chunks_take(L.mem) ? plan.n_long : 0, stepped = plan.n_long + plan.n_short - chunked;
-    if (chunked > 0)
-      if (int rc = memory_chunk_launch(L.mem, in, plan.segs, chunked, cv.row_pos, cache.state, ws.mem_o, s->max_mem, st)) return rc;
+    if (chunked > 0) {
+      if (int rc = reserve_chunks(m, plan.n_chunks)) return rc;
+      const MemoryChunks k{plan.segs, plan.chunks, plan.chunk0, chunked, plan.n_chunks, s->mem_U, s->mem_meta};
+      if (int rc = memory_chunk_launch(L.mem, in, k, cv.row_pos, cache.state, ws.mem_o, s->max_mem, st)) return rc;
+    }
     if (stepped > 0)
       if (int rc = memory_step_launch(L.mem, in, plan.segs + chunked, stepped, cv.row_pos, cache.state, ws.mem_o, s->max_mem, st))
         return rc;
@@ -968,7 +990,7 @@ void layered_destroy(b200_model *m) {
   release(s->many.owned);
   release(s->owned);
   cudaFree(s->x_want); cudaFree(s->h_want); cudaFree(s->logits); cudaFree(s->want); cudaFree(s->next);
-  cudaFree(s->keys16); cudaFree(s->kv16);
+  cudaFree(s->keys16); cudaFree(s->kv16); cudaFree(s->mem_U); cudaFree(s->mem_meta);
   delete s;
   m->lay = nullptr;
 }
@@ -1104,6 +1126,18 @@ static int make_plan(LayeredWs &ws, const std::vector<RowSegment> &segs, bool de
         quad(g.row0 + r, std::min(kHeadsQueryTile, g.n - r), g.seq, g.pos0 + r);
         plan->n_tiles += 1;
       }
+  const size_t chunks = h.size();
+  std::vector<int32_t> chunk0;
+  for (const RowSegment &g : segs)
+    if (is_long(g)) {
+      chunk0.push_back(plan->n_chunks);
+      for (int r = 0; r < g.n; r += kMemoryChunk) {
+        quad(g.row0 + r, std::min(kMemoryChunk, g.n - r), g.seq, g.pos0 + r);
+        plan->n_chunks += 1;
+      }
+    }
+  const size_t firsts = h.size();
+  h.insert(h.end(), chunk0.begin(), chunk0.end());
   const size_t singles = h.size();
   if (dense_rows)
     for (const RowSegment &g : segs)
@@ -1114,6 +1148,8 @@ static int make_plan(LayeredWs &ws, const std::vector<RowSegment> &segs, bool de
   B200_CUDA(cudaMemcpyAsync(ws.plan, h.data(), h.size() * 4, cudaMemcpyHostToDevice, st));   // pageable: copied before it returns
   plan->segs = (const int4 *)ws.plan;
   plan->tiles = (const int4 *)(ws.plan + tiles);
+  plan->chunks = (const int4 *)(ws.plan + chunks);
+  plan->chunk0 = ws.plan + firsts;
   plan->singles = ws.plan + singles;
   return B200_OK;
 }

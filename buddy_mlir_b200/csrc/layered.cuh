@@ -180,7 +180,17 @@ bool memory_chunks_take(const MemoryDims &d);
 // n segments (first row, rows, slot, -) of consecutive tokens; o: [row][ldo]
 int memory_step_launch(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, const int32_t *row_pos, float *states,
                        float *o, int64_t ldo, cudaStream_t st);
-int memory_chunk_launch(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, const int32_t *row_pos, float *states,
+// n_segs segments in chunks of kMemoryChunk rows (first row, rows, slot, -); chunk0: the first chunk of a
+// segment.  U [chunk][head][head_state] and meta [chunk][head][3]: scratch.
+constexpr int kMemoryChunk = 64;
+struct MemoryChunks {
+  const int4 *segs, *chunks;
+  const int32_t *chunk0;
+  int n_segs, n_chunks;
+  float *U;
+  double *meta;
+};
+int memory_chunk_launch(const MemoryDims &d, const MemoryIn &in, const MemoryChunks &k, const int32_t *row_pos, float *states,
                         float *o, int64_t ldo, cudaStream_t st);
 
 // The output projection's input rows from attention shares and / or memory outputs (heads.cu).

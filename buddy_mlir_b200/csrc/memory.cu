@@ -5,12 +5,14 @@
 // and S = n = 0, m = 0 before the first token (position 0 ignores what the slot holds).
 //
 //   memory_step_kernel   token by token, f32: a CTA keeps 32 columns of S in registers
-//   memory_chunk_kernel  64 tokens at a time on mma.sync.  With F the running sum of f inside the
-//                        chunk, a_s = i_s - F_s and M_t = max(m, max_{s<=t} a_s), unrolling gives
-//                          num_t = exp(m - M_t) S^T q_t + sum_{s<=t} exp(a_s - M_t) (q_t k_s) v_s
-//                        and m_t = F_t + M_t: three products per chunk.  q, k, v are the bfloat16
-//                        projections; S, the gated scores and the gated values enter as two bf16
-//                        terms and are summed in f32; F and a are kept in double.
+//   long runs of tokens in chunks of 64, all chunks at once, on mma.sync.  With F the running sum of
+//   f inside a chunk, a_s = i_s - F_s and M_t = max(m, max_{s<=t} a_s), unrolling gives
+//     num_t = exp(m - M_t) S^T q_t + sum_{s<=t} exp(a_s - M_t) (q_t k_s) v_s,   m_t = F_t + M_t
+//     memory_update_kernel  a chunk's own contribution U = sum_s exp(a_s - max a) k_s [v_s | 1]
+//     memory_carry_kernel   S, n, m through the chunks of a segment: U becomes the state before each
+//     memory_read_kernel    the outputs of a chunk from the state before it
+//   q, k, v are the bfloat16 projections; S, the gated scores and the gated values enter the products
+//   as two bf16 terms and are summed in f32; F, a and m are kept in double.
 //
 // State of a slot, per head: S [dim][tiles * 32], then for each 32-column tile its own copy of
 // n [dim], then of m, so that the CTAs of a head need nothing from one another.  m is a sum of as
@@ -109,290 +111,369 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
     store_max(sM, m);
 }
 
-constexpr int kChunk = 64;
+constexpr int kChunk = kMemoryChunk;
+static_assert(kChunk == 64, "two tokens per lane, sixteen per warp");
 
-// grid (segments * heads, columns / VT), 4 warps
+// The gates of a chunk by one warp, two tokens per lane: F, a, and the maximum of a up to the
+// lane's second token; tokens from n on add nothing.
+__device__ __forceinline__ void gate_scan(const MemoryDims &d, const MemoryIn &in, const float *p0, int n, int h, int lane,
+                                          double (&F)[2], double (&a)[2], double &best) {
+  double f[2];
+  float ig[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int t = 2 * lane + i;
+    const float *p = p0 + (int64_t)min(t, n - 1) * in.ldp;
+    ig[i] = capped(p[in.off_i + h], d.cap);
+    f[i] = t < n ? (double)log_sigmoid(capped(p[in.off_f + h], d.cap)) : 0.0;
+  }
+  double sum = f[0] + f[1];
+#pragma unroll
+  for (int w = 1; w < 32; w <<= 1) {
+    const double u = __shfl_up_sync(0xffffffffu, sum, w);
+    if (lane >= w)
+      sum += u;
+  }
+  F[0] = sum - f[1];
+  F[1] = sum;
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+    a[i] = 2 * lane + i < n ? (double)ig[i] - F[i] : -1e300;
+  best = fmax(a[0], a[1]);
+#pragma unroll
+  for (int w = 1; w < 32; w <<= 1) {
+    const double u = __shfl_up_sync(0xffffffffu, best, w);
+    if (lane >= w)
+      best = fmax(best, u);
+  }
+}
+
+// elements c .. c + 3 of a row part of `width` elements (zero from there on); vec: 16-byte loads
+__device__ __forceinline__ float4 load4(const float *p, int c, int width, bool vec) {
+  if (vec && c + 3 < width)
+    return *reinterpret_cast<const float4 *>(p + c);
+  return make_float4(c < width ? p[c] : 0.f, c + 1 < width ? p[c + 1] : 0.f, c + 2 < width ? p[c + 2] : 0.f,
+                     c + 3 < width ? p[c + 3] : 0.f);
+}
+__device__ __forceinline__ void put4(bf16 *dst, const float4 &v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2 *>(dst) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+__device__ __forceinline__ void put4_split(bf16 *hi, bf16 *lo, const float4 &v) {
+  uint32_t h[2], l[2];
+  split2(v.x, v.y, h[0], l[0]);
+  split2(v.z, v.w, h[1], l[1]);
+  *reinterpret_cast<uint2 *>(hi) = make_uint2(h[0], h[1]);
+  *reinterpret_cast<uint2 *>(lo) = make_uint2(l[0], l[1]);
+}
+// rows [n][width] of a projection part as bf16 [kChunk][LK] columns 0 .. DK - 1, zero beyond
+template <int DK>
+__device__ __forceinline__ void load_rows(bf16 *dst, const float *src, int64_t ldp, int n, int width, float factor, bool vec) {
+  for (int i = threadIdx.x; i < kChunk * (DK / 4); i += 128) {
+    const int r = i / (DK / 4), c = 4 * (i - r * (DK / 4));
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < n)
+      v = load4(src + (int64_t)r * ldp, c, width, vec);
+    put4(dst + r * (DK + 8) + c, make_float4(v.x * factor, v.y * factor, v.z * factor, v.w * factor));
+  }
+}
+// VT columns of the values from column v0 on, then a column of ones: elements c .. c + 3 of row r
+template <int VT>
+__device__ __forceinline__ float4 value4(const MemoryDims &d, const float *row, int v0, int c, bool live, bool vec) {
+  if (!live)
+    return make_float4(0.f, 0.f, 0.f, 0.f);
+  if (c >= VT)
+    return make_float4(c == VT ? 1.f : 0.f, 0.f, 0.f, 0.f);
+  return load4(row + v0, c, d.vdim - v0, vec);
+}
+
+// grid (chunks * heads, columns / VT), 4 warps: a warp computes DK / 4 rows of U
 template <int DK, int VT>
 __global__ void __launch_bounds__(128)
-memory_chunk_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, const int32_t *row_pos, float *states, float *o,
-                    int64_t ldo) {
+memory_update_kernel(const MemoryDims d, const MemoryIn in, const int4 *chunks, float *U, double *meta) {
   constexpr int L = kChunk, LK = DK + 8, VA = VT + 8, LV = VA + 8, NT = VA / 8, MT = DK / 64;
+  extern __shared__ __align__(16) bf16 smc[];
+  bf16 *s_k = smc;                                 // [L][LK]
+  bf16 *s_wh = s_k + L * LK, *s_wl = s_wh + L * LV;   // gated [v | 1], two terms
+  __shared__ float s_w[L];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int chunk = blockIdx.x / d.heads, h = blockIdx.x - chunk * d.heads, v0 = blockIdx.y * VT;
+  const int4 seg = chunks[chunk];
+  const int n = seg.y;
+  const float *p0 = in.proj + (int64_t)seg.x * in.ldp;
+  if (warp == 0) {
+    double F[2], a[2], best;
+    gate_scan(d, in, p0, n, h, lane, F, a, best);
+    const double A = __shfl_sync(0xffffffffu, best, 31);
+    s_w[2 * lane] = expf((float)(a[0] - A));
+    s_w[2 * lane + 1] = expf((float)(a[1] - A));
+    if (lane == 31 && blockIdx.y == 0) {
+      meta[(int64_t)blockIdx.x * 3] = A;
+      meta[(int64_t)blockIdx.x * 3 + 1] = F[1];
+    }
+  }
+  load_rows<DK>(s_k, p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, 1.f, (d.dim & 3) == 0);
+  __syncthreads();
+  for (int i = tid; i < L * (LV / 4); i += 128) {
+    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
+    // the values as the bf16 they are elsewhere, times the gate
+    const float4 v = value4<VT>(d, p0 + (int64_t)r * in.ldp + in.off_v + h * d.vdim, v0, c, r < n, (d.vdim & 3) == 0);
+    const float w = s_w[r];
+    auto g = [&](float x) { return __bfloat162float(__float2bfloat16_rn(x)) * w; };
+    put4_split(s_wh + r * LV + c, s_wl + r * LV + c, make_float4(g(v.x), g(v.y), g(v.z), g(v.w)));
+  }
+  __syncthreads();
+  float S[MT][NT][4];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+      S[mt][nt][0] = S[mt][nt][1] = S[mt][nt][2] = S[mt][nt][3] = 0.f;
+#pragma unroll
+  for (int kk = 0; kk < L / 16; ++kk)
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      uint32_t a[4];
+      ldsm4t(a, s_k + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + warp * (DK / 4) + mt * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+      for (int nt = 0; nt < NT; nt += 2) {         // the odd last block reads its zero padding along
+        uint32_t b[4];
+        const int at = (kk * 16 + (lane & 15)) * LV + (lane >> 4) * 8 + nt * 8;
+        ldsm4t(b, s_wh + at);
+        mma16816(S[mt][nt], a, b[0], b[1]);
+        if (nt + 1 < NT)
+          mma16816(S[mt][nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
+        ldsm4t(b, s_wl + at);
+        mma16816(S[mt][nt], a, b[0], b[1]);
+        if (nt + 1 < NT)
+          mma16816(S[mt][nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
+      }
+    }
+  const int64_t ld = d.tiles * 32;
+  float *out = U + (int64_t)blockIdx.x * d.head_state;
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        const int r = warp * (DK / 4) + mt * 16 + (lane >> 2) + g * 8, c = nt * 8 + (lane & 3) * 2;
+        if (r >= d.dim)
+          continue;
+        if (c < VT) {
+          if (v0 + c < ld)
+            *reinterpret_cast<float2 *>(out + r * ld + v0 + c) = make_float2(S[mt][nt][2 * g], S[mt][nt][2 * g + 1]);
+        } else if (c == VT && blockIdx.y == 0) {
+          out[d.dim * ld + r] = S[mt][nt][2 * g];
+        }
+      }
+}
+
+// grid (segments * heads, elements of [S | n] / 1024): four elements per thread, through the chunks
+__global__ void __launch_bounds__(256)
+memory_carry_kernel(const MemoryDims d, const int4 *segs, const int32_t *chunk0, const int32_t *row_pos, float *U, double *meta,
+                    float *states) {
+  const int sg = blockIdx.x / d.heads, h = blockIdx.x - sg * d.heads;
+  const int4 seg = segs[sg];
+  const int n = (seg.y + kChunk - 1) / kChunk, c0 = chunk0[sg];
+  const bool fresh = row_pos[seg.x] == 0;
+  float *st = states + (int64_t)seg.z * d.state + (int64_t)h * d.head_state;
+  const int e = (blockIdx.y * 256 + threadIdx.x) * 4, nS = d.dim * d.tiles * 32;
+  const bool live = e < nS + d.dim;
+  float *sM = st + nS + d.tiles * d.dim;
+  double m = fresh ? 0.0 : load_max(sM);
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (!fresh && live)
+    S = e < nS ? *reinterpret_cast<const float4 *>(st + e) : load4(st + nS, e - nS, d.dim, false);
+  float *u = U + ((int64_t)c0 * d.heads + h) * d.head_state + e;
+  double *mt = meta + ((int64_t)c0 * d.heads + h) * 3;
+  const int64_t du = (int64_t)d.heads * d.head_state, dm = (int64_t)d.heads * 3;
+  constexpr int B = 4;
+  for (int c = 0; c < n; c += B) {
+    float4 v[B];
+    double A[B], F[B];
+#pragma unroll
+    for (int i = 0; i < B; ++i)
+      if (c + i < n) {
+        A[i] = mt[(c + i) * dm];
+        F[i] = mt[(c + i) * dm + 1];
+        if (live)
+          v[i] = *reinterpret_cast<const float4 *>(u + (c + i) * du);
+      }
+#pragma unroll
+    for (int i = 0; i < B; ++i)
+      if (c + i < n) {
+        const double M = fmax(m, A[i]);
+        const float keep = expf((float)(m - M)), add = expf((float)(A[i] - M));
+        if (blockIdx.y == 0 && threadIdx.x == 0)
+          mt[(c + i) * dm + 2] = m;
+        if (live) {
+          *reinterpret_cast<float4 *>(u + (c + i) * du) = S;
+          S = make_float4(fmaf(keep, S.x, add * v[i].x), fmaf(keep, S.y, add * v[i].y), fmaf(keep, S.z, add * v[i].z),
+                          fmaf(keep, S.w, add * v[i].w));
+        }
+        m = F[i] + M;
+      }
+  }
+  if (live && e < nS) {
+    *reinterpret_cast<float4 *>(st + e) = S;
+  } else if (live) {
+    const float a[4] = {S.x, S.y, S.z, S.w};
+    for (int t = 0; t < d.tiles; ++t)
+      for (int i = 0; i < 4; ++i)
+        if (e - nS + i < d.dim)
+          st[nS + t * d.dim + e - nS + i] = a[i];
+  }
+}
+
+// grid (chunks * heads, columns / VT), 4 warps of 16 tokens; a segment's last chunk leaves the
+// running maximum in the state (the carry kernel, whose CTAs all read the old one, has ended)
+template <int DK, int VT>
+__global__ void __launch_bounds__(128)
+memory_read_kernel(const MemoryDims d, const MemoryIn in, const int4 *chunks, int n_chunks, const float *U, const double *meta,
+                   float *states, float *o, int64_t ldo) {
+  constexpr int L = kChunk, LK = DK + 8, VA = VT + 8, LV = VA + 8, NT = VA / 8;
   extern __shared__ __align__(16) bf16 smc[];
   bf16 *s_q = smc, *s_k = s_q + L * LK;            // [L][LK]
   bf16 *s_v = s_k + L * LK;                        // [L][LV]: v | 1
-  bf16 *s_wh = s_v + L * LV, *s_wl = s_wh + L * LV;   // gated [v | 1], two terms
-  bf16 *s_sh = s_wl + L * LV, *s_sl = s_sh + DK * LV; // [DK][LV]: [S | n], two terms
-  __shared__ double s_a[L];
-  __shared__ double s_top[L];                      // M_t
-  __shared__ float s_inter[L], s_floor[L], s_w[L], s_keep;
-  __shared__ double s_m;                           // m before the chunk
+  bf16 *s_sh = s_v + L * LV, *s_sl = s_sh + DK * LV;  // [DK][LV]: [S | n], two terms
+  __shared__ double s_a[L], s_top[L];              // a, M
+  __shared__ float s_inter[L], s_floor[L];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int h = blockIdx.x % d.heads, v0 = blockIdx.y * VT;
-  const int4 seg = segs[blockIdx.x / d.heads];
-  float *st = states + (int64_t)seg.z * d.state + (int64_t)h * d.head_state;
-  const int64_t ld = d.tiles * 32;
-  float *sN = st + d.dim * ld, *sM = sN + (int64_t)d.tiles * d.dim;
-  const int tile0 = v0 / 32, tile1 = min(tile0 + VT / 32, d.tiles);
-  const bool fresh = row_pos[seg.x] == 0;
-  // this thread's part of [S | n]: rows warp * DK/4 + 16 mt + (lane >> 2) (+ 8), columns 8 nt + 2 (lane & 3) (+ 1)
-  float S[MT][NT][4];
-  auto each = [&](auto f) {
+  const int chunk = blockIdx.x / d.heads, h = blockIdx.x - chunk * d.heads, v0 = blockIdx.y * VT;
+  const int4 seg = chunks[chunk];
+  const int n = seg.y;
+  const float *p0 = in.proj + (int64_t)seg.x * in.ldp;
+  if (warp == 0) {
+    double F[2], a[2], best;
+    gate_scan(d, in, p0, n, h, lane, F, a, best);
+    const double m0 = meta[(int64_t)blockIdx.x * 3 + 2];
+    double before = __shfl_up_sync(0xffffffffu, best, 1);
+    before = lane == 0 ? m0 : fmax(before, m0);
+    const double top[2] = {fmax(before, a[0]), fmax(before, fmax(a[0], a[1]))};
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          f(S[mt][nt][e], warp * (DK / 4) + mt * 16 + (lane >> 2) + (e >> 1) * 8, nt * 8 + (lane & 3) * 2 + (e & 1));
-  };
-  each([&](float &x, int r, int c) {
-    x = 0.f;
-    if (!fresh && r < d.dim) {
-      if (c < VT && v0 + c < ld)
-        x = st[r * ld + v0 + c];
-      else if (c == VT)
-        x = sN[(int64_t)tile0 * d.dim + r];
+    for (int i = 0; i < 2; ++i) {
+      const int t = 2 * lane + i;
+      s_a[t] = a[i];
+      s_top[t] = top[i];
+      s_inter[t] = expf((float)(m0 - top[i]));
+      s_floor[t] = expf((float)-(F[i] + top[i]));
     }
-  });
-  if (tid == 0)
-    s_m = fresh ? 0.0 : load_max(sM + 2 * tile0);
-  for (int i = tid; i < (2 * L * LK + 3 * L * LV + 2 * DK * LV) / 8; i += 128)
-    reinterpret_cast<uint4 *>(smc)[i] = make_uint4(0, 0, 0, 0);
-  __syncthreads();
-  for (int c0 = 0; c0 < seg.y; c0 += L) {
-    const int n = min(L, seg.y - c0);
-    const float *p0 = in.proj + (int64_t)(seg.x + c0) * in.ldp;
-    // gates: a scan over the chunk by the first warp, two tokens per lane
-    if (warp == 0) {
-      double f[2], a[2], top[2];
-      float ig[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 2 * lane + i;
-        const float *p = p0 + (int64_t)min(t, n - 1) * in.ldp;
-        ig[i] = capped(p[in.off_i + h], d.cap);
-        f[i] = t < n ? (double)log_sigmoid(capped(p[in.off_f + h], d.cap)) : 0.0;
-      }
-      double sum = f[0] + f[1];
-#pragma unroll
-      for (int w = 1; w < 32; w <<= 1) {
-        const double u = __shfl_up_sync(0xffffffffu, sum, w);
-        if (lane >= w)
-          sum += u;
-      }
-      const double F[2] = {sum - f[1], sum};
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-        a[i] = 2 * lane + i < n ? (double)ig[i] - F[i] : -1e300;
-      const double m0 = s_m;
-      double best = fmax(a[0], a[1]);
-#pragma unroll
-      for (int w = 1; w < 32; w <<= 1) {
-        const double u = __shfl_up_sync(0xffffffffu, best, w);
-        if (lane >= w)
-          best = fmax(best, u);
-      }
-      double before = __shfl_up_sync(0xffffffffu, best, 1);
-      before = lane == 0 ? m0 : fmax(before, m0);
-      top[0] = fmax(before, a[0]);
-      top[1] = fmax(top[0], a[1]);
-      const double last = __shfl_sync(0xffffffffu, top[1], 31), Fl = __shfl_sync(0xffffffffu, F[1], 31);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 2 * lane + i;
-        s_a[t] = a[i];
-        s_top[t] = top[i];
-        s_inter[t] = expf((float)(m0 - top[i]));
-        s_floor[t] = expf((float)-(F[i] + top[i]));
-        s_w[t] = expf((float)(a[i] - last));
-      }
-      __syncwarp();
-      if (lane == 0) {
-        s_keep = expf((float)(m0 - last));
-        s_m = Fl + last;
-      }
+    if (lane == 31 && blockIdx.y == 0 && (chunk + 1 == n_chunks || chunks[chunk + 1].z != seg.z)) {
+      float *sM = states + (int64_t)seg.z * d.state + (int64_t)h * d.head_state + (int64_t)d.dim * d.tiles * 32 + d.tiles * d.dim;
+      for (int t = 0; t < d.tiles; ++t)
+        store_max(sM + 2 * t, F[1] + top[1]);
     }
-    // the rows, bf16
-    for (int i = tid; i < L * (DK / 2); i += 128) {
-      const int r = i / (DK / 2), c = 2 * (i - r * (DK / 2));
-      if (c >= d.dim)
-        continue;
-      float2 q = make_float2(0.f, 0.f), k = q;
-      if (r < n) {
-        const float *p = p0 + (int64_t)r * in.ldp + h * d.dim + c;
-        q.x = p[in.off_q] * d.q_scale;
-        k.x = p[in.off_k];
-        if (c + 1 < d.dim) {
-          q.y = p[in.off_q + 1] * d.q_scale;
-          k.y = p[in.off_k + 1];
-        }
-      }
-      *reinterpret_cast<__nv_bfloat162 *>(s_q + r * LK + c) = __floats2bfloat162_rn(q.x, q.y);
-      *reinterpret_cast<__nv_bfloat162 *>(s_k + r * LK + c) = __floats2bfloat162_rn(k.x, k.y);
-    }
-    for (int i = tid; i < L * (VA / 2); i += 128) {
-      const int r = i / (VA / 2), c = 2 * (i - r * (VA / 2));
-      float2 v = make_float2(0.f, 0.f);
-      if (r < n) {
-        const float *p = p0 + (int64_t)r * in.ldp + in.off_v + h * d.vdim + v0 + c;
-        if (c == VT)
-          v.x = 1.f;
-        else if (c < VT) {
-          if (v0 + c < d.vdim) v.x = p[0];
-          if (v0 + c + 1 < d.vdim) v.y = p[1];
-        }
-      }
-      *reinterpret_cast<__nv_bfloat162 *>(s_v + r * LV + c) = __floats2bfloat162_rn(v.x, v.y);
-    }
-    // [S | n] as two terms
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-        for (int g = 0; g < 2; ++g) {
-          const int at = (warp * (DK / 4) + mt * 16 + (lane >> 2) + g * 8) * LV + nt * 8 + (lane & 3) * 2;
-          uint32_t hi, lo;
-          split2(S[mt][nt][2 * g], S[mt][nt][2 * g + 1], hi, lo);
-          *reinterpret_cast<uint32_t *>(s_sh + at) = hi;
-          *reinterpret_cast<uint32_t *>(s_sl + at) = lo;
-        }
-    __syncthreads();
-    // gated values of the update
-    for (int i = tid; i < L * (VA / 2); i += 128) {
-      const int r = i / (VA / 2), c = 2 * (i - r * (VA / 2));
-      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(s_v + r * LV + c));
-      uint32_t hi, lo;
-      split2(v.x * s_w[r], v.y * s_w[r], hi, lo);
-      *reinterpret_cast<uint32_t *>(s_wh + r * LV + c) = hi;
-      *reinterpret_cast<uint32_t *>(s_wl + r * LV + c) = lo;
-    }
-    const int t0 = warp * 16 + (lane >> 2);        // this thread's tokens: t0, t0 + 8
-    if (warp * 16 < n) {
-      float acc[NT][4], s[8][4];
-#pragma unroll
-      for (int i = 0; i < NT; ++i)
-        acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-        s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-#pragma unroll 2
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        uint32_t a[4];
-        ldsm4(a, s_q + (warp * 16 + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt)
-          if (nt <= warp) {                        // tokens after this warp's are not seen
-            uint32_t b[4];
-            ldsm4(b, s_k + (nt * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + kk * 16 + ((lane >> 3) & 1) * 8);
-            mma16816(s[2 * nt], a, b[0], b[1]);
-            mma16816(s[2 * nt + 1], a, b[2], b[3]);
-          }
-        const int at = (kk * 16 + (lane & 15)) * LV + (lane >> 4) * 8;
-#pragma unroll
-        for (int nt = 0; nt < NT; nt += 2) {       // the odd last block reads its zero padding along
-          uint32_t b[4];
-          ldsm4t(b, s_sh + at + nt * 8);
-          mma16816(acc[nt], a, b[0], b[1]);
-          if (nt + 1 < NT)
-            mma16816(acc[nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
-          ldsm4t(b, s_sl + at + nt * 8);
-          mma16816(acc[nt], a, b[0], b[1]);
-          if (nt + 1 < NT)
-            mma16816(acc[nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
-        }
-      }
-      const double top[2] = {s_top[t0], s_top[t0 + 8]};
-      const float inter[2] = {s_inter[t0], s_inter[t0 + 8]};
-#pragma unroll
-      for (int i = 0; i < NT; ++i)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          acc[i][e] *= inter[e >> 1];
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-        if (i < 2 * warp + 2)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int j = i * 8 + (lane & 3) * 2 + (e & 1);
-            s[i][e] = j <= t0 + (e >> 1) * 8 ? s[i][e] * expf((float)(s_a[j] - top[e >> 1])) : 0.f;
-          }
-#pragma unroll
-      for (int kt = 0; kt < 4; ++kt)
-        if (kt <= warp) {
-          uint32_t hi[4], lw[4];
-          split2(s[2 * kt][0], s[2 * kt][1], hi[0], lw[0]);
-          split2(s[2 * kt][2], s[2 * kt][3], hi[1], lw[1]);
-          split2(s[2 * kt + 1][0], s[2 * kt + 1][1], hi[2], lw[2]);
-          split2(s[2 * kt + 1][2], s[2 * kt + 1][3], hi[3], lw[3]);
-#pragma unroll
-          for (int nt = 0; nt < NT; nt += 2) {
-            uint32_t b[4];
-            ldsm4t(b, s_v + (kt * 16 + (lane & 15)) * LV + (lane >> 4) * 8 + nt * 8);
-            mma16816(acc[nt], hi, b[0], b[1]);
-            mma16816(acc[nt], lw, b[0], b[1]);
-            if (nt + 1 < NT) {
-              mma16816(acc[nt + 1 < NT ? nt + 1 : nt], hi, b[2], b[3]);
-              mma16816(acc[nt + 1 < NT ? nt + 1 : nt], lw, b[2], b[3]);
-            }
-          }
-        }
-#pragma unroll
-      for (int g = 0; g < 2; ++g) {
-        const int t = t0 + 8 * g;
-        const float nq = __shfl_sync(0xffffffffu, acc[NT - 1][2 * g], lane & ~3);   // the column of ones
-        if (t >= n)
-          continue;
-        const float inv = 1.0f / (fmaxf(fabsf(nq), s_floor[t]) + d.floor);
-        float *dst = o + (int64_t)(seg.x + c0 + t) * ldo + h * d.vdim + v0;
-#pragma unroll
-        for (int i = 0; i < NT - 1; ++i) {
-          const int c = i * 8 + (lane & 3) * 2;
-          if (v0 + c < d.vdim)
-            dst[c] = acc[i][2 * g] * inv;
-          if (v0 + c + 1 < d.vdim)
-            dst[c + 1] = acc[i][2 * g + 1] * inv;
-        }
-      }
-    }
-    __syncthreads();                               // gated values are complete
-    // [S | n] = keep * [S | n] + K^T [gated v | gate]
-    const float keep = s_keep;
-    each([&](float &x, int, int) { x *= keep; });
-#pragma unroll
-    for (int kk = 0; kk < L / 16; ++kk) {
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        uint32_t a[4];
-        ldsm4t(a, s_k + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + warp * (DK / 4) + mt * 16 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-        for (int nt = 0; nt < NT; nt += 2) {
-          uint32_t b[4];
-          const int at = (kk * 16 + (lane & 15)) * LV + (lane >> 4) * 8 + nt * 8;
-          ldsm4t(b, s_wh + at);
-          mma16816(S[mt][nt], a, b[0], b[1]);
-          if (nt + 1 < NT)
-            mma16816(S[mt][nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
-          ldsm4t(b, s_wl + at);
-          mma16816(S[mt][nt], a, b[0], b[1]);
-          if (nt + 1 < NT)
-            mma16816(S[mt][nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
-        }
-      }
-    }
-    __syncthreads();                               // the next chunk overwrites the operands
   }
-  each([&](float &x, int r, int c) {
+  const bool vec = (d.dim & 3) == 0, vvec = (d.vdim & 3) == 0;
+  load_rows<DK>(s_q, p0 + in.off_q + h * d.dim, in.ldp, n, d.dim, d.q_scale, vec);
+  load_rows<DK>(s_k, p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, 1.f, vec);
+  for (int i = tid; i < L * (LV / 4); i += 128) {
+    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
+    put4(s_v + r * LV + c, value4<VT>(d, p0 + (int64_t)r * in.ldp + in.off_v + h * d.vdim, v0, c, r < n, vvec));
+  }
+  const int64_t ld = d.tiles * 32;
+  const float *S = U + (int64_t)blockIdx.x * d.head_state;
+  for (int i = tid; i < DK * (LV / 4); i += 128) {
+    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (r < d.dim) {
       if (c < VT && v0 + c < ld)
-        st[r * ld + v0 + c] = x;
+        v = *reinterpret_cast<const float4 *>(S + r * ld + v0 + c);
       else if (c == VT)
-        for (int t = tile0; t < tile1; ++t)
-          sN[(int64_t)t * d.dim + r] = x;
+        v.x = S[d.dim * ld + r];
     }
-  });
-  if (tid >= tile0 && tid < tile1)
-    store_max(sM + 2 * tid, s_m);
+    put4_split(s_sh + r * LV + c, s_sl + r * LV + c, v);
+  }
+  __syncthreads();
+  if (warp * 16 >= n)
+    return;
+  const int t0 = warp * 16 + (lane >> 2);          // this thread's tokens: t0, t0 + 8
+  float acc[NT][4], s[8][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+    acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll 2
+  for (int kk = 0; kk < DK / 16; ++kk) {
+    uint32_t a[4];
+    ldsm4(a, s_q + (warp * 16 + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+      if (nt <= warp) {                            // tokens after this warp's are not seen
+        uint32_t b[4];
+        ldsm4(b, s_k + (nt * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + kk * 16 + ((lane >> 3) & 1) * 8);
+        mma16816(s[2 * nt], a, b[0], b[1]);
+        mma16816(s[2 * nt + 1], a, b[2], b[3]);
+      }
+    const int at = (kk * 16 + (lane & 15)) * LV + (lane >> 4) * 8;
+#pragma unroll
+    for (int nt = 0; nt < NT; nt += 2) {
+      uint32_t b[4];
+      ldsm4t(b, s_sh + at + nt * 8);
+      mma16816(acc[nt], a, b[0], b[1]);
+      if (nt + 1 < NT)
+        mma16816(acc[nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
+      ldsm4t(b, s_sl + at + nt * 8);
+      mma16816(acc[nt], a, b[0], b[1]);
+      if (nt + 1 < NT)
+        mma16816(acc[nt + 1 < NT ? nt + 1 : nt], a, b[2], b[3]);
+    }
+  }
+  const double top[2] = {s_top[t0], s_top[t0 + 8]};
+  const float inter[2] = {s_inter[t0], s_inter[t0 + 8]};
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      acc[i][e] *= inter[e >> 1];
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (i < 2 * warp + 2)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = i * 8 + (lane & 3) * 2 + (e & 1);
+        s[i][e] = j <= t0 + (e >> 1) * 8 ? s[i][e] * expf((float)(s_a[j] - top[e >> 1])) : 0.f;
+      }
+#pragma unroll
+  for (int kt = 0; kt < 4; ++kt)
+    if (kt <= warp) {
+      uint32_t hi[4], lw[4];
+      split2(s[2 * kt][0], s[2 * kt][1], hi[0], lw[0]);
+      split2(s[2 * kt][2], s[2 * kt][3], hi[1], lw[1]);
+      split2(s[2 * kt + 1][0], s[2 * kt + 1][1], hi[2], lw[2]);
+      split2(s[2 * kt + 1][2], s[2 * kt + 1][3], hi[3], lw[3]);
+#pragma unroll
+      for (int nt = 0; nt < NT; nt += 2) {
+        uint32_t b[4];
+        ldsm4t(b, s_v + (kt * 16 + (lane & 15)) * LV + (lane >> 4) * 8 + nt * 8);
+        mma16816(acc[nt], hi, b[0], b[1]);
+        mma16816(acc[nt], lw, b[0], b[1]);
+        if (nt + 1 < NT) {
+          mma16816(acc[nt + 1 < NT ? nt + 1 : nt], hi, b[2], b[3]);
+          mma16816(acc[nt + 1 < NT ? nt + 1 : nt], lw, b[2], b[3]);
+        }
+      }
+    }
+#pragma unroll
+  for (int g = 0; g < 2; ++g) {
+    const int t = t0 + 8 * g;
+    const float nq = __shfl_sync(0xffffffffu, acc[NT - 1][2 * g], lane & ~3);   // the column of ones
+    if (t >= n)
+      continue;
+    const float inv = 1.0f / (fmaxf(fabsf(nq), s_floor[t]) + d.floor);
+    float *dst = o + (int64_t)(seg.x + t) * ldo + h * d.vdim + v0;
+#pragma unroll
+    for (int i = 0; i < NT - 1; ++i) {
+      const int c = i * 8 + (lane & 3) * 2;
+      if (v0 + c < d.vdim)
+        dst[c] = acc[i][2 * g] * inv;
+      if (v0 + c + 1 < d.vdim)
+        dst[c + 1] = acc[i][2 * g + 1] * inv;
+    }
+  }
 }
 
 template <int R>
@@ -402,19 +483,33 @@ int step_run(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, c
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
-template <int DK, int VT>
-int chunk_run(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, const int32_t *row_pos, float *states, float *o,
-              int64_t ldo, cudaStream_t st) {
-  const size_t smem = ((size_t)2 * kChunk * (DK + 8) + (size_t)3 * kChunk * (VT + 16) + (size_t)2 * DK * (VT + 16)) * 2;
+template <auto Kern> int allow(size_t bytes) {
   static int configured[64] = {};
   int dev = 0;
   B200_CUDA(cudaGetDevice(&dev));
   if (dev < 0 || dev >= 64 || !configured[dev]) {
-    B200_CUDA(cudaFuncSetAttribute(memory_chunk_kernel<DK, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    B200_CUDA(cudaFuncSetAttribute(Kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
     if (dev >= 0 && dev < 64)
       configured[dev] = 1;
   }
-  memory_chunk_kernel<DK, VT><<<dim3(n * d.heads, (d.tiles * 32 + VT - 1) / VT), 128, smem, st>>>(d, in, segs, row_pos, states, o, ldo);
+  return B200_OK;
+}
+
+template <int DK, int VT>
+int chunk_run(const MemoryDims &d, const MemoryIn &in, const MemoryChunks &k, const int32_t *row_pos, float *states, float *o,
+              int64_t ldo, cudaStream_t st) {
+  constexpr int L = kChunk, LK = DK + 8, LV = VT + 16;
+  const size_t update = ((size_t)L * LK + (size_t)2 * L * LV) * 2;
+  const size_t read = ((size_t)2 * L * LK + (size_t)L * LV + (size_t)2 * DK * LV) * 2;
+  if (int rc = allow<memory_update_kernel<DK, VT>>(update)) return rc;
+  if (int rc = allow<memory_read_kernel<DK, VT>>(read)) return rc;
+  const dim3 grid(k.n_chunks * d.heads, (d.tiles * 32 + VT - 1) / VT);
+  memory_update_kernel<DK, VT><<<grid, 128, update, st>>>(d, in, k.chunks, k.U, k.meta);
+  B200_LAUNCH_CHECK();
+  const int elems = d.dim * d.tiles * 32 + d.dim;
+  memory_carry_kernel<<<dim3(k.n_segs * d.heads, (elems + 1023) / 1024), 256, 0, st>>>(d, k.segs, k.chunk0, row_pos, k.U, k.meta, states);
+  B200_LAUNCH_CHECK();
+  memory_read_kernel<DK, VT><<<grid, 128, read, st>>>(d, in, k.chunks, k.n_chunks, k.U, k.meta, states, o, ldo);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -437,13 +532,13 @@ int memory_step_launch(const MemoryDims &d, const MemoryIn &in, const int4 *segs
   return step_run<64>(d, in, segs, n, row_pos, states, o, ldo, st);
 }
 
-int memory_chunk_launch(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, const int32_t *row_pos, float *states,
+int memory_chunk_launch(const MemoryDims &d, const MemoryIn &in, const MemoryChunks &k, const int32_t *row_pos, float *states,
                         float *o, int64_t ldo, cudaStream_t st) {
   if (d.dim <= 64)
-    return d.vdim <= 32 ? chunk_run<64, 32>(d, in, segs, n, row_pos, states, o, ldo, st) : chunk_run<64, 64>(d, in, segs, n, row_pos, states, o, ldo, st);
+    return d.vdim <= 32 ? chunk_run<64, 32>(d, in, k, row_pos, states, o, ldo, st) : chunk_run<64, 64>(d, in, k, row_pos, states, o, ldo, st);
   if (d.dim <= 128)
-    return chunk_run<128, 32>(d, in, segs, n, row_pos, states, o, ldo, st);
-  return chunk_run<256, 32>(d, in, segs, n, row_pos, states, o, ldo, st);
+    return chunk_run<128, 64>(d, in, k, row_pos, states, o, ldo, st);
+  return chunk_run<256, 32>(d, in, k, row_pos, states, o, ldo, st);
 }
 
 } // namespace b200
