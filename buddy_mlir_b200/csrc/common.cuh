@@ -40,6 +40,27 @@ int ensure_device();
                           cudaGetErrorString(e_), __FILE__, __LINE__);         \
   } while (0)
 
+// ---- chained launches ---------------------------------------------------------
+// A kernel launched by launch_chained may start while the kernel before it in the stream still
+// runs: it calls chain_wait() before it touches anything another kernel writes (or reads), which
+// returns when everything before it has ended.  chain_next() lets the kernel after it start.
+__device__ __forceinline__ void chain_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void chain_next() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+template <typename... P, typename... A>
+inline cudaError_t launch_chained(void (*kern)(P...), dim3 grid, int threads, size_t smem, cudaStream_t st, const A &...args) {
+  cudaLaunchConfig_t c{};
+  c.gridDim = grid;
+  c.blockDim = dim3((unsigned)threads);
+  c.dynamicSmemBytes = smem;
+  c.stream = st;
+  cudaLaunchAttribute a{};
+  a.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  a.val.programmaticStreamSerializationAllowed = 1;
+  c.attrs = &a;
+  c.numAttrs = 1;
+  return cudaLaunchKernelEx(&c, kern, static_cast<P>(args)...);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1)

@@ -135,21 +135,15 @@ __device__ void stage_settled(const RowsP &p, float4 *xs, float *s_red) {
 }
 
 template <typename T, int MT, int R>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, MT == 1 ? 4 : 1)
 gemv_rows_kernel(const RowsP p) {
   extern __shared__ __align__(16) float4 xs[];   // [MT][slab / 4]
   __shared__ float s_r[8], s_red[8];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int m0 = blockIdx.y * MT, rows = min(MT, p.M - m0);
   const float *x = p.x + (int64_t)m0 * p.ldx;
-  {
-    // the CTA's first weight rows start on their way to L2 under the prologue
-    const int64_t row = (int64_t)blockIdx.x * kWarps * R + warp * R + lane;
-    if (lane < R && row < p.N) {
-      const T *w = reinterpret_cast<const T *>(p.w) + row * p.ldw;
-      asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(w), "r"((uint32_t)(unit_pad<T>(p.K) * sizeof(T))) : "memory");
-    }
-  }
+  chain_wait();
+  chain_next();
   const bool settles = MT == 1 && p.x_out != nullptr;
   if (settles)
     stage_settled<T>(p, xs, s_red);
@@ -379,7 +373,7 @@ template <typename T, int MT, int R> int gemv_rows_run(RowsP &p, cudaStream_t st
   const int y = (p.M + MT - 1) / MT;
   int grid = 1;
   if (int rc = wave_grid(kern, (p.N + kWarps * R - 1) / (kWarps * R), y, smem, &grid)) return rc;
-  kern<<<dim3(grid, y), kThreads, smem, st>>>(p);
+  B200_CUDA(launch_chained(kern, dim3(grid, y), kThreads, smem, st, p));
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

@@ -53,6 +53,8 @@ heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const Cach
   extern __shared__ float s_cs[];
   __shared__ float s_red[16];
   const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
+  chain_wait();
+  chain_next();
   const float *src = in.proj + (int64_t)m * in.ldp, *ks = src + in.off_k, *vs = src + in.off_v;
   const int pos = cv.row_pos[m];
   turn_table(s_cs, in.freq, d.rot >> 1, pos, tid, 256);
@@ -124,6 +126,8 @@ heads_attend_kernel(const HeadsDims d, const T *q, const int32_t *rows, const T 
   extern __shared__ float sm[];
   const int g_all = d.heads / d.kv, chunks = (g_all + kGroup - 1) / kGroup;
   const int kvh = blockIdx.y / chunks, g0 = (blockIdx.y - kvh * chunks) * kGroup, g = min(kGroup, g_all - g0);
+  chain_wait();
+  chain_next();
   const int m = rows ? rows[blockIdx.z] : (int)blockIdx.z, h0 = kvh * g_all + g0;
   const int pos = cv.row_pos[m], seq = cv.row_seq[m];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -232,9 +236,13 @@ heads_decode_kernel(const HeadsDims d, const bf16 *q, const int32_t *rows, const
   y /= vchunks;
   const int kvh = y / hchunks, g0 = (y - kvh * hchunks) * 16, g = min(16, g_all - g0), h0 = kvh * g_all + g0;
   const int v0 = vc * DV, nv = min(DV, d.vdimp - v0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int i = tid; i < (16 * LK + 4 * WARP) / 8; i += 128)
+    reinterpret_cast<uint4 *>(smb)[i] = make_uint4(0, 0, 0, 0);
+  chain_wait();
+  chain_next();
   const int m = rows ? rows[blockIdx.z] : (int)blockIdx.z;
   const int pos = cv.row_pos[m], seq = cv.row_seq[m];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   int k0, k1;
   split_range(d, pos, blockIdx.x, gridDim.x, 64, k0, k1);
   if (k0 >= k1) {
@@ -245,8 +253,6 @@ heads_decode_kernel(const HeadsDims d, const bf16 *q, const int32_t *rows, const
     }
     return;
   }
-  for (int i = tid; i < (16 * LK + 4 * WARP) / 8; i += 128)
-    reinterpret_cast<uint4 *>(smb)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
   for (int i = tid; i < g * d.dimp / 8; i += 128) {
     const int r = i / (d.dimp / 8), c = (i - r * (d.dimp / 8)) * 8;
@@ -395,6 +401,8 @@ __global__ void __launch_bounds__(128)
 mix_finish_kernel(const MixFinish f) {
   __shared__ float s_w[kMaxSplits];
   __shared__ float4 s_o[4][32];
+  chain_wait();
+  chain_next();
   const int m = f.rows ? f.rows[blockIdx.x] : (int)blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const CatRow out{f.cat ? f.cat + (int64_t)m * f.ldc : nullptr, f.cat16 ? f.cat16 + (int64_t)m * f.ldc : nullptr};
   const float *proj = f.proj + (int64_t)m * f.ldp;
@@ -696,7 +704,7 @@ int decode_run(const HeadsDims &d, const bf16 *q, const int32_t *rows, int n, co
   if (int rc = allow<heads_decode_kernel<DK, DV>>(smem)) return rc;
   const int g = d.heads / d.kv;
   const dim3 grid(splits, d.kv * ((g + 15) / 16) * ((d.vdimp + DV - 1) / DV), n);
-  heads_decode_kernel<DK, DV><<<grid, 128, smem, st>>>(d, q, rows, pool, cv, part);
+  B200_CUDA(launch_chained(heads_decode_kernel<DK, DV>, grid, 128, smem, st, d, q, rows, pool, cv, part));
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -735,9 +743,9 @@ int heads_prep_launch(int dtype, const HeadsDims &d, const HeadsIn &in, int M, v
   const int units = (d.heads + 2 * d.kv + 7) / 8;
   const dim3 grid(M, std::max(1, std::min(units, 592 / M)));
   if (dtype == B200_F32)
-    heads_prep_kernel<float><<<grid, 256, smem, st>>>(d, in, (float *)q, (float *)pool, cv);
+    B200_CUDA(launch_chained(heads_prep_kernel<float>, grid, 256, smem, st, d, in, (float *)q, (float *)pool, cv));
   else
-    heads_prep_kernel<bf16><<<grid, 256, smem, st>>>(d, in, (bf16 *)q, (bf16 *)pool, cv);
+    B200_CUDA(launch_chained(heads_prep_kernel<bf16>, grid, 256, smem, st, d, in, (bf16 *)q, (bf16 *)pool, cv));
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -758,17 +766,17 @@ int heads_attend_launch(int dtype, const HeadsDims &d, const void *q, const int3
   const size_t smem = (size_t)kGroup * (d.dimp + d.vdimp + kTile) * 4;
   if (dtype == B200_F32) {
     if (int rc = allow<heads_attend_kernel<float>>(smem)) return rc;
-    heads_attend_kernel<float><<<grid, 128, smem, st>>>(d, (const float *)q, rows, (const float *)pool, cv, part);
+    B200_CUDA(launch_chained(heads_attend_kernel<float>, grid, 128, smem, st, d, (const float *)q, rows, (const float *)pool, cv, part));
   } else {
     if (int rc = allow<heads_attend_kernel<bf16>>(smem)) return rc;
-    heads_attend_kernel<bf16><<<grid, 128, smem, st>>>(d, (const bf16 *)q, rows, (const bf16 *)pool, cv, part);
+    B200_CUDA(launch_chained(heads_attend_kernel<bf16>, grid, 128, smem, st, d, (const bf16 *)q, rows, (const bf16 *)pool, cv, part));
   }
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
 
 int mix_finish_launch(const MixFinish &f, int M, cudaStream_t st) {
-  mix_finish_kernel<<<dim3(M, f.n_heads + (f.n_mem + 3) / 4), 128, 0, st>>>(f);
+  B200_CUDA(launch_chained(mix_finish_kernel, dim3(M, f.n_heads + (f.n_mem + 3) / 4), 128, 0, st, f));
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

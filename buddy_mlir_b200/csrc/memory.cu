@@ -44,6 +44,8 @@ memory_step_kernel(const MemoryDims d, const MemoryIn in, const int4 *segs, cons
   __shared__ float s_q[2][DM], s_k[2][DM], s_o[2][8][32], s_n[2][8];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h = blockIdx.x % d.heads, tile = blockIdx.y, col = tile * 32 + lane;
+  chain_wait();
+  chain_next();
   const int4 seg = segs[blockIdx.x / d.heads];     // first row, rows, slot
   float *st = states + (int64_t)seg.z * d.state + (int64_t)h * d.head_state;
   float *sS = st + col, *sN = st + (int64_t)d.dim * d.tiles * 32 + (int64_t)tile * d.dim;
@@ -479,7 +481,7 @@ memory_read_kernel(const MemoryDims d, const MemoryIn in, const int4 *chunks, in
 template <int R>
 int step_run(const MemoryDims &d, const MemoryIn &in, const int4 *segs, int n, const int32_t *row_pos, float *states, float *o,
              int64_t ldo, cudaStream_t st) {
-  memory_step_kernel<R><<<dim3(n * d.heads, d.tiles), 256, 0, st>>>(d, in, segs, row_pos, states, o, ldo);
+  B200_CUDA(launch_chained(memory_step_kernel<R>, dim3(n * d.heads, d.tiles), 256, 0, st, d, in, segs, row_pos, states, o, ldo));
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
