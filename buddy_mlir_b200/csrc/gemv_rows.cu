@@ -89,9 +89,71 @@ __device__ __forceinline__ float cta_sum(float s, float *s_red) {
   return t;
 }
 
+// The same with the row in registers, four groups of four elements per thread (K % 4 == 0).
+constexpr int kRowGroups = 4;
+template <typename T>
+__device__ void stage_settled_short(const RowsP &p, float4 *xs, float *s_red) {
+  float4 x[kRowGroups], y[kRowGroups];
+  const int groups = p.K >> 2;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < kRowGroups; ++i) {
+    const int g = threadIdx.x + i * kThreads;
+    x[i] = g < groups ? reinterpret_cast<const float4 *>(p.x)[g] : zero;
+    y[i] = g < groups && p.late.y != nullptr ? reinterpret_cast<const float4 *>(p.late.y)[g] : zero;
+  }
+  float r = 0.f;
+  if (p.late.y != nullptr) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRowGroups; ++i)
+      s = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, s))));
+    r = 1.0f / sqrtf(cta_sum(s, s_red) / (float)p.K + p.eps);
+  }
+  const T *emb = p.late.embed != nullptr ? reinterpret_cast<const T *>(p.late.embed) + (int64_t)p.late.tokens[0] * p.late.lde : nullptr;
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < kRowGroups; ++i) {
+    const int g = threadIdx.x + i * kThreads;
+    if (g >= groups)
+      continue;
+    float4 &v = x[i];
+    if (p.late.y != nullptr) {
+      const float4 w = __ldg(reinterpret_cast<const float4 *>(p.late.w) + g);
+      v.x = fmaf(y[i].x * r, w.x, v.x); v.y = fmaf(y[i].y * r, w.y, v.y);
+      v.z = fmaf(y[i].z * r, w.z, v.z); v.w = fmaf(y[i].w * r, w.w, v.w);
+    }
+    if (emb != nullptr) {
+      v.x = fmaf(to_float(emb[4 * g]), p.late.scale, v.x); v.y = fmaf(to_float(emb[4 * g + 1]), p.late.scale, v.y);
+      v.z = fmaf(to_float(emb[4 * g + 2]), p.late.scale, v.z); v.w = fmaf(to_float(emb[4 * g + 3]), p.late.scale, v.w);
+    }
+    if (blockIdx.x == 0)
+      reinterpret_cast<float4 *>(p.x_out)[g] = v;
+    s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+  }
+  const float rx = p.norm_w != nullptr ? 1.0f / sqrtf(cta_sum(s, s_red) / (float)p.K + p.eps) : 1.f;
+#pragma unroll
+  for (int i = 0; i < kRowGroups; ++i) {
+    const int g = threadIdx.x + i * kThreads;
+    if (g >= block_pad<T>(p.K) / 4)
+      continue;
+    float4 v = x[i];
+    if (p.norm_w != nullptr && g < groups) {
+      const float4 w = __ldg(reinterpret_cast<const float4 *>(p.norm_w) + g);
+      v = make_float4(v.x * rx * w.x, v.y * rx * w.y, v.z * rx * w.z, v.w * rx * w.w);
+    }
+    xs[stage_slot<T>(g)] = v;                      // zero beyond K
+  }
+  __syncthreads();
+}
+
 // Stage the settled (and normed) row in xs; the first CTA writes the settled row to x_out.
 template <typename T>
 __device__ void stage_settled(const RowsP &p, float4 *xs, float *s_red) {
+  if ((p.K & 3) == 0 && block_pad<T>(p.K) <= 4 * kRowGroups * kThreads) {
+    stage_settled_short<T>(p, xs, s_red);
+    return;
+  }
   float r = 0.f;
   if (p.late.y != nullptr) {
     float s = 0.f;
@@ -142,6 +204,21 @@ gemv_rows_kernel(const RowsP p) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int m0 = blockIdx.y * MT, rows = min(MT, p.M - m0);
   const float *x = p.x + (int64_t)m0 * p.ldx;
+  if (MT == 1) {
+    // while the kernel ahead ends: the norm weights and the beginnings of the CTA's first weight
+    // rows, which nothing writes, on their way to L2
+    for (int k = threadIdx.x * 32; k < p.K; k += kThreads * 32) {
+      if (p.norm_w != nullptr)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(p.norm_w + k));
+      if (p.late.y != nullptr)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(p.late.w + k));
+    }
+    constexpr int kLines = 32 / R;                 // of 128 bytes, per row
+    const int64_t row = (int64_t)blockIdx.x * kWarps * R + warp * R + lane / kLines;
+    const int k = lane % kLines * (128 / (int)sizeof(T));
+    if (row < p.N && k < p.K)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const T *>(p.w) + row * p.ldw + k));
+  }
   chain_wait();
   chain_next();
   const bool settles = MT == 1 && p.x_out != nullptr;
