@@ -150,12 +150,13 @@ __device__ __forceinline__ void gate_scan(const MemoryDims &d, const MemoryIn &i
   }
 }
 
-// elements c .. c + 3 of a row part of `width` elements (zero from there on); vec: 16-byte loads
+// elements c .. c + 3 of a row part of `width` elements (zero from there on); vec: 16-byte loads.
+// Read-only for the whole kernel, so that a thread's loads can all be under way at once.
 __device__ __forceinline__ float4 load4(const float *p, int c, int width, bool vec) {
   if (vec && c + 3 < width)
-    return *reinterpret_cast<const float4 *>(p + c);
-  return make_float4(c < width ? p[c] : 0.f, c + 1 < width ? p[c + 1] : 0.f, c + 2 < width ? p[c + 2] : 0.f,
-                     c + 3 < width ? p[c + 3] : 0.f);
+    return __ldg(reinterpret_cast<const float4 *>(p + c));
+  return make_float4(c < width ? __ldg(p + c) : 0.f, c + 1 < width ? __ldg(p + c + 1) : 0.f, c + 2 < width ? __ldg(p + c + 2) : 0.f,
+                     c + 3 < width ? __ldg(p + c + 3) : 0.f);
 }
 __device__ __forceinline__ void put4(bf16 *dst, const float4 &v) {
   const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
@@ -168,25 +169,40 @@ __device__ __forceinline__ void put4_split(bf16 *hi, bf16 *lo, const float4 &v) 
   *reinterpret_cast<uint2 *>(hi) = make_uint2(h[0], h[1]);
   *reinterpret_cast<uint2 *>(lo) = make_uint2(l[0], l[1]);
 }
-// rows [n][width] of a projection part as bf16 [kChunk][LK] columns 0 .. DK - 1, zero beyond
-template <int DK>
-__device__ __forceinline__ void load_rows(bf16 *dst, const float *src, int64_t ldp, int n, int width, float factor, bool vec) {
-  for (int i = threadIdx.x; i < kChunk * (DK / 4); i += 128) {
-    const int r = i / (DK / 4), c = 4 * (i - r * (DK / 4));
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < n)
-      v = load4(src + (int64_t)r * ldp, c, width, vec);
-    put4(dst + r * (DK + 8) + c, make_float4(v.x * factor, v.y * factor, v.z * factor, v.w * factor));
+// use(row, column, elements column .. column + 3) for every group of four columns 0 .. COLS - 1 of
+// rows 0 .. ROWS - 1 of src; zero from row n and column `width` on.  Eight loads per thread are under
+// way at a time (vec: 16-byte ones; then width % 4 == 0).
+template <int ROWS, int COLS, typename F>
+__device__ __forceinline__ void each4(const float *src, int64_t ld, int n, int width, bool vec, F use) {
+  constexpr int G = COLS / 4, N = ROWS * G, B = 8;
+  static_assert(N % 128 == 0, "whole rounds of 128 threads");
+  if (!vec) {
+    for (int i = threadIdx.x; i < N; i += 128) {
+      const int r = i / G, c = 4 * (i - r * G);
+      use(r, c, r < n ? load4(src + (int64_t)r * ld, c, width, false) : make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+    return;
+  }
+#pragma unroll 1
+  for (int i0 = threadIdx.x; i0 < N; i0 += B * 128) {
+    float4 v[B];
+#pragma unroll
+    for (int j = 0; j < B; ++j) {
+      const int i = i0 + j * 128, r = i / G, c = 4 * (i - r * G);   // beyond the end: some row that exists
+      v[j] = __ldg(reinterpret_cast<const float4 *>(src + (int64_t)min(r, n - 1) * ld + min(c, width - 4)));
+    }
+#pragma unroll
+    for (int j = 0; j < B; ++j) {
+      const int i = i0 + j * 128, r = i / G, c = 4 * (i - r * G);
+      if (i < N)
+        use(r, c, r < n && c < width ? v[j] : make_float4(0.f, 0.f, 0.f, 0.f));
+    }
   }
 }
-// VT columns of the values from column v0 on, then a column of ones: elements c .. c + 3 of row r
-template <int VT>
-__device__ __forceinline__ float4 value4(const MemoryDims &d, const float *row, int v0, int c, bool live, bool vec) {
-  if (!live)
-    return make_float4(0.f, 0.f, 0.f, 0.f);
-  if (c >= VT)
-    return make_float4(c == VT ? 1.f : 0.f, 0.f, 0.f, 0.f);
-  return load4(row + v0, c, d.vdim - v0, vec);
+// the column of ones behind VT value columns, and zeros to the end of the row: use(row, column, elements)
+template <int VT, typename F> __device__ __forceinline__ void each_one(int n, F use) {
+  for (int i = threadIdx.x; i < kChunk * 4; i += 128)
+    use(i >> 2, VT + 4 * (i & 3), make_float4((i & 3) == 0 && (i >> 2) < n ? 1.f : 0.f, 0.f, 0.f, 0.f));
 }
 
 // grid (chunks * heads, columns / VT), 4 warps: a warp computes DK / 4 rows of U
@@ -214,16 +230,16 @@ memory_update_kernel(const MemoryDims d, const MemoryIn in, const int4 *chunks, 
       meta[(int64_t)blockIdx.x * 3 + 1] = F[1];
     }
   }
-  load_rows<DK>(s_k, p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, 1.f, (d.dim & 3) == 0);
+  const bool vec = (d.dim & 3) == 0, vvec = (d.vdim & 3) == 0;
+  each4<L, DK>(p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, vec, [&](int r, int c, const float4 &v) { put4(s_k + r * LK + c, v); });
   __syncthreads();
-  for (int i = tid; i < L * (LV / 4); i += 128) {
-    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
-    // the values as the bf16 they are elsewhere, times the gate
-    const float4 v = value4<VT>(d, p0 + (int64_t)r * in.ldp + in.off_v + h * d.vdim, v0, c, r < n, (d.vdim & 3) == 0);
+  auto put = [&](int r, int c, const float4 &v) {  // the values as the bf16 they are elsewhere, times the gate
     const float w = s_w[r];
     auto g = [&](float x) { return __bfloat162float(__float2bfloat16_rn(x)) * w; };
     put4_split(s_wh + r * LV + c, s_wl + r * LV + c, make_float4(g(v.x), g(v.y), g(v.z), g(v.w)));
-  }
+  };
+  each4<L, VT>(p0 + in.off_v + h * d.vdim + v0, in.ldp, n, d.vdim - v0, vvec, put);
+  each_one<VT>(n, put);
   __syncthreads();
   float S[MT][NT][4];
 #pragma unroll
@@ -285,8 +301,15 @@ memory_carry_kernel(const MemoryDims d, const int4 *segs, const int32_t *chunk0,
   float *sM = st + nS + d.tiles * d.dim;
   double m = fresh ? 0.0 : load_max(sM);
   float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (!fresh && live)
-    S = e < nS ? *reinterpret_cast<const float4 *>(st + e) : load4(st + nS, e - nS, d.dim, false);
+  if (!fresh && live) {
+    if (e < nS) {
+      S = *reinterpret_cast<const float4 *>(st + e);
+    } else {
+      const float *p = st + e;                     // n, the first tile's copy
+      const int w = d.dim - (e - nS);
+      S = make_float4(p[0], w > 1 ? p[1] : 0.f, w > 2 ? p[2] : 0.f, w > 3 ? p[3] : 0.f);
+    }
+  }
   float *u = U + ((int64_t)c0 * d.heads + h) * d.head_state + e;
   double *mt = meta + ((int64_t)c0 * d.heads + h) * 3;
   const int64_t du = (int64_t)d.heads * d.head_state, dm = (int64_t)d.heads * 3;
@@ -368,24 +391,19 @@ memory_read_kernel(const MemoryDims d, const MemoryIn in, const int4 *chunks, in
     }
   }
   const bool vec = (d.dim & 3) == 0, vvec = (d.vdim & 3) == 0;
-  load_rows<DK>(s_q, p0 + in.off_q + h * d.dim, in.ldp, n, d.dim, d.q_scale, vec);
-  load_rows<DK>(s_k, p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, 1.f, vec);
-  for (int i = tid; i < L * (LV / 4); i += 128) {
-    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
-    put4(s_v + r * LV + c, value4<VT>(d, p0 + (int64_t)r * in.ldp + in.off_v + h * d.vdim, v0, c, r < n, vvec));
-  }
-  const int64_t ld = d.tiles * 32;
+  const float qs = d.q_scale;
+  each4<L, DK>(p0 + in.off_q + h * d.dim, in.ldp, n, d.dim, vec,
+               [&](int r, int c, const float4 &v) { put4(s_q + r * LK + c, make_float4(v.x * qs, v.y * qs, v.z * qs, v.w * qs)); });
+  each4<L, DK>(p0 + in.off_k + h * d.dim, in.ldp, n, d.dim, vec, [&](int r, int c, const float4 &v) { put4(s_k + r * LK + c, v); });
+  auto put = [&](int r, int c, const float4 &v) { put4(s_v + r * LV + c, v); };
+  each4<L, VT>(p0 + in.off_v + h * d.vdim + v0, in.ldp, n, d.vdim - v0, vvec, put);
+  each_one<VT>(n, put);
+  const int ld = d.tiles * 32;
   const float *S = U + (int64_t)blockIdx.x * d.head_state;
-  for (int i = tid; i < DK * (LV / 4); i += 128) {
-    const int r = i / (LV / 4), c = 4 * (i - r * (LV / 4));
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < d.dim) {
-      if (c < VT && v0 + c < ld)
-        v = *reinterpret_cast<const float4 *>(S + r * ld + v0 + c);
-      else if (c == VT)
-        v.x = S[d.dim * ld + r];
-    }
-    put4_split(s_sh + r * LV + c, s_sl + r * LV + c, v);
+  each4<DK, VT>(S + v0, ld, d.dim, ld - v0, true, [&](int r, int c, const float4 &v) { put4_split(s_sh + r * LV + c, s_sl + r * LV + c, v); });
+  for (int i = tid; i < DK * 4; i += 128) {
+    const int r = i >> 2, c = VT + 4 * (i & 3);
+    put4_split(s_sh + r * LV + c, s_sl + r * LV + c, make_float4((i & 3) == 0 && r < d.dim ? __ldg(S + d.dim * ld + r) : 0.f, 0.f, 0.f, 0.f));
   }
   __syncthreads();
   if (warp * 16 >= n)
