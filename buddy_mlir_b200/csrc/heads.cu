@@ -46,11 +46,48 @@ __device__ __forceinline__ float turned(const HeadsDims &d, const float *x, int 
   return (c & 1) ? at(c) * cs[i] + at(c - 1) * cs[half + i] : at(c) * cs[i] - at(c + 1) * cs[half + i];
 }
 
+__device__ __forceinline__ void put2(float *p, float a, float b) { *reinterpret_cast<float2 *>(p) = make_float2(a, b); }
+__device__ __forceinline__ void put2(bf16 *p, float a, float b) { *reinterpret_cast<__nv_bfloat162 *>(p) = __floats2bfloat162_rn(a, b); }
+__device__ __forceinline__ float2 get2(const float *x, const float *w, int c, float r) {
+  float2 v = *reinterpret_cast<const float2 *>(x + c);
+  if (w != nullptr) {
+    const float2 n = __ldg(reinterpret_cast<const float2 *>(w + c));
+    v.x *= r * n.x;
+    v.y *= r * n.y;
+  }
+  return v;
+}
+// A head by one warp, two elements at a time (dim even, and rot / 2 for split halves).
+template <typename T>
+__device__ __forceinline__ void turn_head(const HeadsDims &d, const float *x, float r, const float *w, const float *cs, T *dst, int lane) {
+  const int half = d.rot >> 1;
+  if (d.halves) {
+#pragma unroll 2
+    for (int i = 2 * lane; i < half; i += 64) {
+      const float2 u = get2(x, w, i, r), v = get2(x, w, i + half, r);
+      const float2 c = *reinterpret_cast<const float2 *>(cs + i), n = *reinterpret_cast<const float2 *>(cs + half + i);
+      put2(dst + i, u.x * c.x - v.x * n.x, u.y * c.y - v.y * n.y);
+      put2(dst + half + i, v.x * c.x + u.x * n.x, v.y * c.y + u.y * n.y);
+    }
+  } else {
+#pragma unroll 2
+    for (int i = lane; i < half; i += 32) {
+      const float2 v = get2(x, w, 2 * i, r);
+      put2(dst + 2 * i, v.x * cs[i] - v.y * cs[half + i], v.y * cs[i] + v.x * cs[half + i]);
+    }
+  }
+#pragma unroll 2
+  for (int c = d.rot + 2 * lane; c < d.dim; c += 64) {
+    const float2 v = get2(x, w, c, r);
+    put2(dst + c, v.x, v.y);
+  }
+}
+
 // grid (M, y): a row's query, key and value heads are dealt to the warps of its y CTAs
 template <typename T>
 __global__ void __launch_bounds__(256)
 heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const CacheView cv) {
-  extern __shared__ float s_cs[];
+  extern __shared__ __align__(16) float s_cs[];
   __shared__ float s_red[16];
   const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
   chain_wait();
@@ -62,12 +99,22 @@ heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const Cach
   if (in.q_norm != nullptr) {
     const int nq = d.heads * d.dim, nk = d.kv * d.dim;
     float a = 0.f, b = 0.f;
+    auto squares = [tid](const float *x, int n) {
+      float t = 0.f;
+      if ((n & 3) == 0) {
 #pragma unroll 4
-    for (int i = tid; i < nq; i += 256)
-      a = fmaf(src[i], src[i], a);
-#pragma unroll 4
-    for (int i = tid; i < nk; i += 256)
-      b = fmaf(ks[i], ks[i], b);
+        for (int i = tid; i < n / 4; i += 256) {
+          const float4 v = reinterpret_cast<const float4 *>(x)[i];
+          t = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, t))));
+        }
+      } else {
+        for (int i = tid; i < n; i += 256)
+          t = fmaf(x[i], x[i], t);
+      }
+      return t;
+    };
+    a = squares(src, nq);
+    b = squares(ks, nk);
     a = warp_sum(a);
     b = warp_sum(b);
     if (lane == 0) {
@@ -85,22 +132,38 @@ heads_prep_kernel(const HeadsDims d, const HeadsIn in, T *q, T *pool, const Cach
   }
   __syncthreads();
   T *row = pool + cache_row(cv, cv.row_seq[m], pos) * d.row;
+  const bool twos = (d.dim & 1) == 0 && (d.vdim & 1) == 0 && (!d.halves || (d.rot & 3) == 0);
   for (int u = blockIdx.y * 8 + (tid >> 5); u < d.heads + 2 * d.kv; u += gridDim.y * 8) {
-    if (u < d.heads) {
-      T *dst = q + ((int64_t)m * d.heads + u) * d.dimp;
-#pragma unroll 4
-      for (int c = lane; c < d.dimp; c += 32)
-        dst[c] = from_float<T>(c < d.dim ? turned(d, src + u * d.dim, c, rq, in.q_norm ? in.q_norm + u * d.dim : nullptr, s_cs) : 0.f);
-    } else if (u < d.heads + d.kv) {
-      const int h = u - d.heads;
-#pragma unroll 4
-      for (int c = lane; c < d.dim; c += 32)
-        row[h * d.dimp + c] = from_float<T>(turned(d, ks + h * d.dim, c, rk, in.k_norm ? in.k_norm + h * d.dim : nullptr, s_cs));
+    if (u < d.heads + d.kv) {                      // a query or a key head
+      const bool query = u < d.heads;
+      const int h = query ? u : u - d.heads;
+      const float *x = (query ? src : ks) + h * d.dim, *w = query ? in.q_norm : in.k_norm;
+      const float r = query ? rq : rk;
+      T *dst = query ? q + ((int64_t)m * d.heads + h) * d.dimp : row + h * d.dimp;
+      if (w != nullptr)
+        w += h * d.dim;
+      if (twos) {
+        turn_head(d, x, r, w, s_cs, dst, lane);
+      } else {
+        for (int c = lane; c < d.dim; c += 32)
+          dst[c] = from_float<T>(turned(d, x, c, r, w, s_cs));
+      }
+      if (query && d.dim + lane < d.dimp)          // a cache row's padding is zero already
+        dst[d.dim + lane] = from_float<T>(0.f);
     } else {
       const int h = u - d.heads - d.kv;
-#pragma unroll 4
-      for (int c = lane; c < d.vdim; c += 32)
-        row[d.kv * d.dimp + h * d.vdimp + c] = from_float<T>(vs[h * d.vdim + c]);
+      const float *x = vs + h * d.vdim;
+      T *dst = row + d.kv * d.dimp + h * d.vdimp;
+      if (twos) {
+#pragma unroll 2
+        for (int c = 2 * lane; c < d.vdim; c += 64) {
+          const float2 v = *reinterpret_cast<const float2 *>(x + c);
+          put2(dst + c, v.x, v.y);
+        }
+      } else {
+        for (int c = lane; c < d.vdim; c += 32)
+          dst[c] = from_float<T>(x[c]);
+      }
     }
   }
 }
@@ -469,13 +532,34 @@ mix_finish_kernel(const MixFinish f) {
   const int vd = f.mem_vdim;
   const float *o = f.mem_o + (int64_t)m * f.ldo + h * vd;
   float s = 0.f;
-#pragma unroll 4
+  const float *g = proj + f.off_mg + h * vd, *nw = f.mem_norm + h * vd;
+  if ((vd & 3) == 0) {
+#pragma unroll 2
+    for (int c = 4 * lane; c < vd; c += 128) {
+      const float4 v = *reinterpret_cast<const float4 *>(o + c);
+      s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+    }
+    const float r = f.m_scale / sqrtf(warp_sum(s) / (float)vd + f.eps);
+#pragma unroll 2
+    for (int c = 4 * lane; c < vd; c += 128) {
+      const float4 v = *reinterpret_cast<const float4 *>(o + c), z = *reinterpret_cast<const float4 *>(g + c);
+      const float4 w = __ldg(reinterpret_cast<const float4 *>(nw + c));
+      const float4 a = make_float4(gated(v.x * r * w.x, &z.x), gated(v.y * r * w.y, &z.y), gated(v.z * r * w.z, &z.z), gated(v.w * r * w.w, &z.w));
+      const int64_t at = f.mem_col + h * vd + c;
+      if (out.f != nullptr) {
+        *reinterpret_cast<float4 *>(out.f + at) = a;
+      } else {
+        put2(out.b + at, a.x, a.y);
+        put2(out.b + at + 2, a.z, a.w);
+      }
+    }
+    return;
+  }
   for (int c = lane; c < vd; c += 32)
     s = fmaf(o[c], o[c], s);
   const float r = f.m_scale / sqrtf(warp_sum(s) / (float)vd + f.eps);
-#pragma unroll 4
   for (int c = lane; c < vd; c += 32)
-    out.set(f.mem_col + h * vd + c, gated(o[c] * r * f.mem_norm[h * vd + c], proj + f.off_mg + h * vd + c));
+    out.set(f.mem_col + h * vd + c, gated(o[c] * r * nw[c], g + c));
 }
 
 struct FlashP {
@@ -663,7 +747,7 @@ heads_prefill_kernel(const FlashP p) {
 template <typename T>
 __global__ void __launch_bounds__(256)
 heads_shift_kernel(const HeadsDims d, const T *cache, int src, const double *freq, int delta, T *stage) {
-  extern __shared__ float s_cs[];
+  extern __shared__ __align__(16) float s_cs[];
   const int half = d.rot >> 1;
   turn_table(s_cs, freq, half, delta, threadIdx.x, 256);
   __syncthreads();
